@@ -5,6 +5,7 @@ from .sagizen import SagizenConfig
 from .vosulorn import VosulornConfig
 from .redenex import RedenexConfig
 from .radupel import RadupelConfig
+from .sarizen import SarizenConfig
 
 __all__ = ["ConfigError", "LayerSpec", "ModelPlan", "PartSpec", "ScheduleEntry", "config_class_for", "read_config",
-           "register_architecture", "registered_architectures", "LlamaConfig", "SagizenConfig", "VosulornConfig", "RedenexConfig", "RadupelConfig"]
+           "register_architecture", "registered_architectures", "LlamaConfig", "SagizenConfig", "VosulornConfig", "RedenexConfig", "RadupelConfig", "SarizenConfig"]

@@ -38,8 +38,9 @@ __device__ __forceinline__ void angle_sincos(double pos, double f, float* sn, fl
   sincosf((float)a, sn, cs);
 }
 
-// element i (< rot) of a rotated run x[0 .. rot): pairs (2j, 2j + 1) if `interleaved`, else (j, j + rot / 2)
-__device__ __forceinline__ float rotated(const float* x, int i, int rot, int interleaved, double pos, const double* __restrict__ freq) {
+// element i (< rot) of a rotated run x[0 .. rot): pairs (2j, 2j + 1) if `interleaved`, else (j, j + rot / 2); sine and cosine are
+// multiplied by `mult` (1: a plain rotation; stretched rotations may lengthen the rotated part as well)
+__device__ __forceinline__ float rotated(const float* x, int i, int rot, int interleaved, double pos, const double* __restrict__ freq, float mult) {
   const int half = rot >> 1;
   int j, partner;
   bool first;
@@ -47,6 +48,8 @@ __device__ __forceinline__ float rotated(const float* x, int i, int rot, int int
   else { first = i < half; j = first ? i : i - half; partner = first ? i + half : i - half; }
   float sn, cs;
   angle_sincos(pos, freq[j], &sn, &cs);
+  sn *= mult;
+  cs *= mult;
   return first ? x[i] * cs - x[partner] * sn : x[i] * cs + x[partner] * sn;
 }
 
@@ -77,7 +80,7 @@ rotate_append_kernel(const float* __restrict__ qkv, const float* __restrict__ bi
                      const int32_t* __restrict__ tok_pos, const int32_t* __restrict__ tok_seq, const int32_t* __restrict__ page_table,
                      int table_stride, int n_pages, T* __restrict__ kcache, T* __restrict__ vcache, int H, int G, int dk, int dv,
                      int rot, int interleaved, const double* __restrict__ freq, int* __restrict__ err, int maps,
-                     const float* __restrict__ q_norm, const float* __restrict__ k_norm, float eps, int ldq, ConvAhead conv) {
+                     const float* __restrict__ q_norm, const float* __restrict__ k_norm, float eps, int ldq, ConvAhead conv, float mult) {
   pdl_launch_dependents();
   pdl_wait();
   extern __shared__ float ra_stage[];   // MA_WARPS rows of dk floats
@@ -133,7 +136,7 @@ rotate_append_kernel(const float* __restrict__ qkv, const float* __restrict__ bi
     }
     for (int i = lane; i < dk; i += 32) {
       const int mp = i / ds, j = i - mp * ds;
-      const float x = j < rot ? rotated(sh + mp * ds, j, rot, interleaved, (double)pos, freq) : sh[i];
+      const float x = j < rot ? rotated(sh + mp * ds, j, rot, interleaved, (double)pos, freq, mult) : sh[i];
       if (head < H) q_out[((size_t)t * H + head) * dk + i] = x;
       else kcache[(((size_t)page * G + (head - H)) * PAGE + in_page) * dk + i] = from_f32<T>(x);
     }
@@ -148,7 +151,7 @@ rotate_append_kernel(const float* __restrict__ qkv, const float* __restrict__ bi
 }
 
 // u [tokens][ldu] float32: H query heads of [d | rd] from column 0 and, with `has_kv`, the latent's row [r | rd] from
-// column kv_off.  The rotated part of every query head (half-split pairs) goes to q_out[t][h * q_pitch + q_off + i], and with
+// column kv_off.  The rotated part of every query head (pairs and `mult` as in `rotated`) goes to q_out[t][h * q_pitch + q_off + i], and with
 // `copy_q` the unrotated part to q_out[t][h * q_pitch + i]; the latent, divided by its root mean square and times `norm_w`,
 // and the rotated shared key part become the token's cache row [r + rd] (one key head) and, if `row_out` is given, row t
 // of it as well (what the cache holds, for a step that expands its own keys).
@@ -158,7 +161,7 @@ latent_prepare_kernel(const float* __restrict__ u, int ldu, int kv_off, int has_
                       int copy_q, const float* __restrict__ norm_w, float eps, const int32_t* __restrict__ tok_pos,
                       const int32_t* __restrict__ tok_seq, const int32_t* __restrict__ page_table, int table_stride, int n_pages,
                       T* __restrict__ kcache, T* __restrict__ row_out, int H, int d, int rd, int r, const double* __restrict__ freq,
-                      int* __restrict__ err) {
+                      int* __restrict__ err, int interleaved, float mult) {
   pdl_launch_dependents();
   pdl_wait();
   __shared__ float red[33];
@@ -172,7 +175,7 @@ latent_prepare_kernel(const float* __restrict__ u, int ldu, int kv_off, int has_
   float* qo = q_out + (size_t)t * H * q_pitch;
   for (int i = threadIdx.x; i < H * rd; i += blockDim.x) {
     const int h = i / rd, j = i - h * rd;
-    qo[(size_t)h * q_pitch + q_off + j] = rotated(row + (size_t)h * (d + rd) + d, j, rd, 0, (double)pos, freq);
+    qo[(size_t)h * q_pitch + q_off + j] = rotated(row + (size_t)h * (d + rd) + d, j, rd, interleaved, (double)pos, freq, mult);
   }
   if (copy_q)
     for (int i = threadIdx.x; i < H * d; i += blockDim.x) {
@@ -193,7 +196,7 @@ latent_prepare_kernel(const float* __restrict__ u, int ldu, int kv_off, int has_
   T* dst = kcache + ((size_t)page * PAGE + pos % PAGE) * (r + rd);
   T* dst2 = row_out ? row_out + (size_t)t * (r + rd) : nullptr;
   for (int i = threadIdx.x; i < r + rd; i += blockDim.x) {
-    const T v = from_f32<T>(i < r ? c[i] * inv * norm_w[i] : rotated(c + r, i - r, rd, 0, (double)pos, freq));
+    const T v = from_f32<T>(i < r ? c[i] * inv * norm_w[i] : rotated(c + r, i - r, rd, interleaved, (double)pos, freq, mult));
     dst[i] = v;
     if (dst2) dst2[i] = v;
   }
@@ -693,7 +696,8 @@ extern "C" int edgelm_rotate_append(const float* qkv, const float* bias, float* 
                                     const int32_t* page_table, int table_stride, int n_pages, void* kcache, void* vcache, int dtype,
                                     int n_tokens, int H, int G, int dk, int dv, int rot, int interleaved, const double* freq, int* err,
                                     int maps, const float* q_norm, const float* k_norm, float eps, int ldq, const float* conv_w, int taps,
-                                    float* conv_state, const int32_t* seq_tok0, const int32_t* seq_slot, int move_tail, cudaStream_t stream) {
+                                    float* conv_state, const int32_t* seq_tok0, const int32_t* seq_slot, int move_tail, float mult,
+                                    cudaStream_t stream) {
   if (n_tokens == 0) return 0;
   EL_REFUSE(conv_w == nullptr || (taps >= 1 && seq_tok0 != nullptr && seq_slot != nullptr && (taps == 1 || conv_state != nullptr)),
             "rotate_append: a filter of %d taps needs the sequences' first rows, their slots and the tails", taps);
@@ -710,10 +714,10 @@ extern "C" int edgelm_rotate_append(const float* qkv, const float* bias, float* 
   const int bit = pdl_bit_for_tokens(n_tokens);
   if (dtype == DT_F32)
     launch_pdl(bit, rotate_append_kernel<float>, grid, block, smem, stream, qkv, bias, q_out, tok_pos, tok_seq, page_table, table_stride,
-               n_pages, (float*)kcache, (float*)vcache, H, G, dk, dv, rot, interleaved, freq, err, maps, q_norm, k_norm, eps, ldq, conv);
+               n_pages, (float*)kcache, (float*)vcache, H, G, dk, dv, rot, interleaved, freq, err, maps, q_norm, k_norm, eps, ldq, conv, mult);
   else if (dtype == DT_BF16)
     launch_pdl(bit, rotate_append_kernel<__nv_bfloat16>, grid, block, smem, stream, qkv, bias, q_out, tok_pos, tok_seq, page_table,
-               table_stride, n_pages, (__nv_bfloat16*)kcache, (__nv_bfloat16*)vcache, H, G, dk, dv, rot, interleaved, freq, err, maps, q_norm, k_norm, eps, ldq, conv);
+               table_stride, n_pages, (__nv_bfloat16*)kcache, (__nv_bfloat16*)vcache, H, G, dk, dv, rot, interleaved, freq, err, maps, q_norm, k_norm, eps, ldq, conv, mult);
   else
     EL_REFUSE(false, "rotate_append: unknown dtype code %d", dtype);
   EL_LAUNCH_CHECK("rotate_append");
@@ -723,7 +727,8 @@ extern "C" int edgelm_rotate_append(const float* qkv, const float* bias, float* 
 extern "C" int edgelm_latent_prepare(const float* u, int ldu, int kv_off, int has_kv, float* q_out, int q_pitch, int q_off, int copy_q,
                                      const float* norm_w, float eps, const int32_t* tok_pos, const int32_t* tok_seq,
                                      const int32_t* page_table, int table_stride, int n_pages, void* kcache, void* row_out, int dtype,
-                                     int n_tokens, int H, int d, int rd, int r, const double* freq, int* err, cudaStream_t stream) {
+                                     int n_tokens, int H, int d, int rd, int r, const double* freq, int* err, int interleaved, float mult,
+                                     cudaStream_t stream) {
   if (n_tokens == 0) return 0;
   EL_REFUSE(n_tokens > 0 && H > 0 && d >= 0 && r >= 1 && rd >= 0 && rd % 2 == 0, "latent_prepare: sizes heads %d, %d + %d, latent %d", H, d, rd, r);
   EL_REFUSE(rd == 0 || freq != nullptr, "latent_prepare: no frequencies");
@@ -732,11 +737,11 @@ extern "C" int edgelm_latent_prepare(const float* u, int ldu, int kv_off, int ha
   const int bit = pdl_bit_for_tokens(n_tokens);
   if (dtype == DT_F32)
     launch_pdl(bit, latent_prepare_kernel<float>, dim3(n_tokens), dim3(256), (size_t)0, stream, u, ldu, kv_off, has_kv, q_out, q_pitch, q_off, copy_q,
-               norm_w, eps, tok_pos, tok_seq, page_table, table_stride, n_pages, (float*)kcache, (float*)row_out, H, d, rd, r, freq, err);
+               norm_w, eps, tok_pos, tok_seq, page_table, table_stride, n_pages, (float*)kcache, (float*)row_out, H, d, rd, r, freq, err, interleaved, mult);
   else if (dtype == DT_BF16)
     launch_pdl(bit, latent_prepare_kernel<__nv_bfloat16>, dim3(n_tokens), dim3(256), (size_t)0, stream, u, ldu, kv_off, has_kv, q_out, q_pitch, q_off,
                copy_q, norm_w, eps, tok_pos, tok_seq, page_table, table_stride, n_pages, (__nv_bfloat16*)kcache, (__nv_bfloat16*)row_out, H, d, rd,
-               r, freq, err);
+               r, freq, err, interleaved, mult);
   else
     EL_REFUSE(false, "latent_prepare: unknown dtype code %d", dtype);
   EL_LAUNCH_CHECK("latent_prepare");

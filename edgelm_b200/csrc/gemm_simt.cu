@@ -7,6 +7,7 @@
 //   EPI_STORE     out[M, N] (float or bfloat16)             = acc
 //   EPI_RESIDUAL  out[M, N] (float) = residual[M, N] + acc   (out may be residual itself)
 //   EPI_SWIGLU    out[M, N] = silu(acc_gate) * acc_up with a second weight W2 (up) of W's shape
+//   EPI_RELU2     out[M, N] = max(acc, 0)^2
 // Two kernels: a 64x64 tile for many rows and a one-warp-per-output-column kernel for a few
 // rows (decode), which reads every weight once.  Each output element is summed over k in an
 // order that depends on K alone, never on M or on the row's place in the batch.
@@ -14,7 +15,7 @@
 
 namespace edgelm {
 
-enum : int { EPI_STORE = 0, EPI_RESIDUAL = 1, EPI_SWIGLU = 2 };
+enum : int { EPI_STORE = 0, EPI_RESIDUAL = 1, EPI_SWIGLU = 2, EPI_RELU2 = 4 };
 
 __device__ __forceinline__ float silu_f32(float z) { return z / (1.0f + expf(-z)); }
 
@@ -23,6 +24,7 @@ __device__ __forceinline__ void epilogue_store(TOut* out, const float* residual,
   if (EPI == EPI_STORE) out[idx] = from_f32<TOut>(acc);
   if (EPI == EPI_RESIDUAL) out[idx] = from_f32<TOut>(residual[idx] + acc);
   if (EPI == EPI_SWIGLU) out[idx] = from_f32<TOut>(silu_f32(acc) * acc2);
+  if (EPI == EPI_RELU2) out[idx] = from_f32<TOut>(fmaxf(acc, 0.f) * fmaxf(acc, 0.f));
 }
 
 // ------------------------------------------------------------------ tiled kernel
@@ -206,6 +208,7 @@ extern "C" int edgelm_gemm_simt(const void* a, int lda, const void* w, const voi
     case EPI_STORE: launch_gemm<TA, TA, EPI_STORE, TOUT>(a, lda, w, w2, out, ldo, residual, M, N, K, force_kernel, stream); break;       \
     case EPI_RESIDUAL: launch_gemm<TA, TA, EPI_RESIDUAL, float>(a, lda, w, w2, out, ldo, residual, M, N, K, force_kernel, stream); break; \
     case EPI_SWIGLU: launch_gemm<TA, TA, EPI_SWIGLU, TOUT>(a, lda, w, w2, out, ldo, residual, M, N, K, force_kernel, stream); break;     \
+    case EPI_RELU2: launch_gemm<TA, TA, EPI_RELU2, TOUT>(a, lda, w, w2, out, ldo, residual, M, N, K, force_kernel, stream); break;       \
     default: EL_REFUSE(false, "gemm_simt: unknown epilogue %d", epilogue);                                           \
   }
   if (a_dtype == DT_F32 && out_dtype == DT_F32) {

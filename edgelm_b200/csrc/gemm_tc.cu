@@ -23,7 +23,8 @@
 
 namespace edgelm {
 
-enum : int { TC_EPI_STORE = 0, TC_EPI_RESIDUAL = 1, TC_EPI_SWIGLU = 2, TC_EPI_ROPE = 3 };
+// (TC_EPI_RELU2 is the store epilogue with `RopeAppend::square_relu` set: no kernel of its own is compiled for it)
+enum : int { TC_EPI_STORE = 0, TC_EPI_RESIDUAL = 1, TC_EPI_SWIGLU = 2, TC_EPI_ROPE = 3, TC_EPI_RELU2 = 4 };
 
 // What the epilogue of the stacked q, k, v projection of a prompt step needs to finish the job of three kernels
 // (TC_EPI_ROPE): each token's position, its sequence's row of the page table, the rotation table, the cache.
@@ -43,6 +44,11 @@ struct RopeAppend {
   // g = min(gate, limit), v = clamp(up, -limit, limit) + shift; limit 0: no clamps (alpha 1, shift 0: SwiGLU)
   float glu_limit = 0.f, glu_alpha = 1.f, glu_shift = 0.f;
   const float* glu_bias = nullptr;   // [2 N] float32 (gate's | up's), added to the two sums before the unit; null: none
+  int square_relu = 0;               // the store epilogue writes max(sum, 0)^2
+  // grouped products: row r holds pair row_pair[r] (negative: none), whose weight multiplies both sums before the unit, as if the
+  // row of `a` had been multiplied by it (no rounding of that product to bfloat16 in between); pair_weight null: no weights
+  const int32_t* row_pair = nullptr;
+  const float* pair_weight = nullptr;
 };
 
 // Grouped products (a feed-forward of experts): the rows of `a` come grouped, every group's rows starting at a multiple of
@@ -115,7 +121,7 @@ __device__ __forceinline__ void fetch_residual(ResidualAhead& ra, const float* r
 template <int EPI, typename TOut>
 __device__ __forceinline__ void epilogue_piece(const uint32_t* r, const uint32_t* r2, TOut* out, int ldo,
                                                const float* residual, int row, int col0, int M, int N, int vec_ok,
-                                               const RopeAppend& form, const ResidualAhead* ahead = nullptr) {
+                                               const RopeAppend& form, const ResidualAhead* ahead = nullptr, float row_weight = 1.f) {
   if (row >= M) return;
   const size_t base = (size_t)row * ldo + col0;
   const bool full = vec_ok && (col0 + 32 <= N);
@@ -126,13 +132,16 @@ __device__ __forceinline__ void epilogue_piece(const uint32_t* r, const uint32_t
     for (int j = 0; j < 8; ++j) {
       const float acc = __uint_as_float(r[j0 + j]);
       if (EPI == TC_EPI_SWIGLU) {
-        float g = acc, u = __uint_as_float(r2[j0 + j]);
+        float g = acc * row_weight, u = __uint_as_float(r2[j0 + j]) * row_weight;
         if (form.glu_bias != nullptr) {     // (every thread of a tile asks for the same 2 x 32 values: they come out of L1)
           const int c = min(col0 + j0 + j, N - 1);
           g += form.glu_bias[c];
           u += form.glu_bias[N + c];
         }
         v[j] = glu_tc(g, u, form.glu_limit, form.glu_alpha, form.glu_shift);
+      } else if (EPI == TC_EPI_STORE && form.square_relu) {
+        const float z = fmaxf(acc, 0.f);
+        v[j] = z * z;
       } else v[j] = acc;
     }
     if (full) {
@@ -383,6 +392,11 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
     if (EPI == TC_EPI_RESIDUAL && k_splits == 1) fetch_residual(ra[0], residual, ldo, m0 + q * 32 + lane, n0, M, N, vec_ok);  // while the MMAs run
     RopeRow rr;
     if constexpr (EPI == TC_EPI_ROPE) rope_row_fetch(rr, rope, m0 + q * 32 + lane, M, n0 + BN > rope.nh * rope.hd, err);   // likewise
+    float row_weight = 1.f;
+    if (EPI == TC_EPI_SWIGLU && rope.pair_weight != nullptr && m0 + q * 32 + lane < M) {   // likewise
+      const int pair = rope.row_pair[m0 + q * 32 + lane];
+      row_weight = pair >= 0 ? rope.pair_weight[pair] : 0.f;
+    }
     const bool ok = __all_sync(0xffffffffu, mbar_wait(smem_u32(tmem_full_bar), 0, abort_flag, err));  // one decision per warp
     asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
     if (ok && EPI == TC_EPI_ROPE) {
@@ -419,7 +433,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
           }
           continue;
         }
-        epilogue_piece<EPI, TOut>(r, r2, out, ldo, residual, m0 + q * 32 + lane, n0 + c0, M, N, vec_ok, rope, &ra[(c0 >> 5) & 1]);
+        epilogue_piece<EPI, TOut>(r, r2, out, ldo, residual, m0 + q * 32 + lane, n0 + c0, M, N, vec_ok, rope, &ra[(c0 >> 5) & 1], row_weight);
       }
     }
   }
@@ -434,7 +448,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
 // out = epilogue(sum over the splits, in their order, of the raw sums a split-K launch left).
 template <int EPI, typename TOut>
 __global__ void splitk_reduce_kernel(const float* __restrict__ partial, int splits, TOut* out, int ldo, const float* residual,
-                                     int M, int N, float glu_limit, float glu_alpha, float glu_shift, const float* __restrict__ glu_bias) {
+                                     int M, int N, float glu_limit, float glu_alpha, float glu_shift, const float* __restrict__ glu_bias, int square_relu) {
   constexpr int NB = EPI == TC_EPI_SWIGLU ? 2 : 1;
   const size_t plane = (size_t)M * N;
   for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < plane; i += (size_t)gridDim.x * blockDim.x) {
@@ -447,6 +461,7 @@ __global__ void splitk_reduce_kernel(const float* __restrict__ partial, int spli
     const size_t o = (size_t)m * ldo + n;
     if (EPI == TC_EPI_SWIGLU) out[o] = from_f32<TOut>(glu_tc(a + (glu_bias ? glu_bias[n] : 0.f), b + (glu_bias ? glu_bias[N + n] : 0.f), glu_limit, glu_alpha, glu_shift));
     else if (EPI == TC_EPI_RESIDUAL) out[o] = from_f32<TOut>(residual[o] + a);
+    else if (square_relu) out[o] = from_f32<TOut>(fmaxf(a, 0.f) * fmaxf(a, 0.f));
     else out[o] = from_f32<TOut>(a);
   }
 }
@@ -706,7 +721,7 @@ static int launch_tc(const CUtensorMap& ma, const CUtensorMap& mb, const CUtenso
   if (EPI != TC_EPI_ROPE && splits > 1) {
     const size_t plane = (size_t)M * N;
     const int blocks = (int)((plane + 255) / 256 < 1184 ? (plane + 255) / 256 : 1184);
-    splitk_reduce_kernel<EPI, TOut><<<blocks, 256, 0, stream>>>(g_splitk_ws, splits, (TOut*)out, ldo, residual, M, N, rope.glu_limit, rope.glu_alpha, rope.glu_shift, rope.glu_bias);
+    splitk_reduce_kernel<EPI, TOut><<<blocks, 256, 0, stream>>>(g_splitk_ws, splits, (TOut*)out, ldo, residual, M, N, rope.glu_limit, rope.glu_alpha, rope.glu_shift, rope.glu_bias, rope.square_relu);
   }
   return 0;
 }
@@ -859,18 +874,22 @@ extern "C" int edgelm_gemm_tc_glu(const void* a, int lda, const void* w, const v
 extern "C" int edgelm_gemm_tc(const void* a, int lda, const void* w, const void* w2, void* out, int ldo,
                               const float* residual, int M, int N, int K, int out_dtype, int epilogue, int* err,
                               cudaStream_t stream) {
-  EL_REFUSE(epilogue >= TC_EPI_STORE && epilogue <= TC_EPI_SWIGLU, "gemm_tc: unknown epilogue %d", epilogue);
-  return gemm_tc_run(a, lda, w, w2, out, ldo, residual, M, N, K, out_dtype, epilogue, err, stream, RopeAppend{});
+  EL_REFUSE((epilogue >= TC_EPI_STORE && epilogue <= TC_EPI_SWIGLU) || epilogue == TC_EPI_RELU2, "gemm_tc: unknown epilogue %d", epilogue);
+  RopeAppend form{};
+  form.square_relu = epilogue == TC_EPI_RELU2;
+  return gemm_tc_run(a, lda, w, w2, out, ldo, residual, M, N, K, out_dtype, epilogue == TC_EPI_RELU2 ? TC_EPI_STORE : epilogue, err, stream, form);
 }
 
 // A grouped product: a [M, K] with M a multiple of 128 (rows grouped, every group's first row at a multiple of 128),
 // w [n_groups * N, K] the groups' weights stacked; row tile t uses group tile_group[t] (negative: no rows).  out [M, N].
 // Epilogues: store (float32 or bfloat16) and the gated unit (w2 the second stacked weight, bfloat16 out; its form as in
-// `edgelm_gemm_tc_glu`: limit 0, alpha 1, shift 0 is SwiGLU).
+// `edgelm_gemm_tc_glu`: limit 0, alpha 1, shift 0 is SwiGLU).  With `pair_weight` (and `row_pair` [M]) the gated unit's two sums of row r
+// are multiplied by pair_weight[row_pair[r]] first (0 for a row of no pair): the weight on the input of a group's product.
 extern "C" int edgelm_gemm_tc_grouped(const void* a, int lda, const void* w, const void* w2, void* out, int ldo, int M, int N, int K,
                                       int n_groups, const int32_t* tile_group, int out_dtype, int epilogue, float glu_limit, float glu_alpha,
-                                      float glu_shift, int* err, cudaStream_t stream) {
+                                      float glu_shift, const int32_t* row_pair, const float* pair_weight, int* err, cudaStream_t stream) {
   if (M == 0) return 0;
+  EL_REFUSE(pair_weight == nullptr || (row_pair != nullptr && epilogue == TC_EPI_SWIGLU), "gemm_tc_grouped: weights need the rows' pairs and the gated unit");
   EL_REFUSE(M > 0 && M % TC_BM == 0 && N > 0 && K > 0 && n_groups > 0 && lda >= K && ldo >= N && tile_group != nullptr, "gemm_tc_grouped: bad sizes M=%d N=%d K=%d groups=%d", M, N, K, n_groups);
   EL_REFUSE(edgelm_gemm_tc_takes(a, lda, w, w2, K), "gemm_tc_grouped: K=%d and lda=%d must be multiples of 8 and the operands 16-byte aligned", K, lda);
   EL_REFUSE((epilogue == TC_EPI_SWIGLU && w2 != nullptr && out_dtype == DT_BF16) || epilogue == TC_EPI_STORE, "gemm_tc_grouped: epilogue %d with output dtype %d", epilogue, out_dtype);
@@ -891,6 +910,8 @@ extern "C" int edgelm_gemm_tc_grouped(const void* a, int lda, const void* w, con
   form.glu_limit = glu_limit;
   form.glu_alpha = glu_alpha;
   form.glu_shift = glu_shift;
+  form.row_pair = row_pair;
+  form.pair_weight = pair_weight;
   if (epilogue == TC_EPI_SWIGLU)
     rc = launch_tc<64, TC_EPI_SWIGLU, __nv_bfloat16>(ma, mb, mb2, out, ldo, nullptr, M, N, K, vec_ok, err, stream, false, form, grp);
   else if (out_dtype == DT_F32)

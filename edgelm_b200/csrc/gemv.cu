@@ -10,7 +10,7 @@
 //     stand-alone norm kernel rounds it), which removes a kernel and a round trip per use;
 //   * each warp's first weight loads are issued before the prologue, so that memory latency and
 //     the prologue overlap;
-//   * epilogues as everywhere: store, += residual (float32), SwiGLU of two weights.
+//   * epilogues as everywhere: store, += residual (float32), SwiGLU of two weights, squared ReLU.
 // A column's sum is taken in an order that depends on K alone (lane-strided partial sums, then
 // a fixed shuffle tree), so a row's result does not depend on the rest of the batch.
 // Takes K a multiple of the 16-byte vector (8 bfloat16, 4 float) with aligned rows; other
@@ -19,7 +19,7 @@
 
 namespace edgelm {
 
-enum : int { GV_STORE = 0, GV_RESIDUAL = 1, GV_SWIGLU = 2 };
+enum : int { GV_STORE = 0, GV_RESIDUAL = 1, GV_SWIGLU = 2, GV_RELU2 = 4 };
 constexpr int GV_ROWS = 8;
 
 template <typename T> struct Vec16;
@@ -228,6 +228,7 @@ gemv_kernel(const T* __restrict__ act, int lda, const float* __restrict__ x, con
           if (EPI == GV_STORE) out[idx] = from_f32<TOut>(s);
           if (EPI == GV_RESIDUAL) out[idx] = from_f32<TOut>(res + s);
           if (EPI == GV_SWIGLU) out[idx] = from_f32<TOut>(gv_silu(s) * s2);
+          if (EPI == GV_RELU2) out[idx] = from_f32<TOut>(fmaxf(s, 0.f) * fmaxf(s, 0.f));
         }
       }
     }
@@ -307,12 +308,14 @@ extern "C" int edgelm_gemv(const void* act, int lda, const float* norm_w, float 
     else if (epilogue == GV_STORE && out_dtype == DT_F32) rc = EL_GV(__nv_bfloat16, GV_STORE, float);
     else if (epilogue == GV_RESIDUAL) rc = EL_GV(__nv_bfloat16, GV_RESIDUAL, float);
     else if (epilogue == GV_SWIGLU && out_dtype == DT_BF16) rc = EL_GV(__nv_bfloat16, GV_SWIGLU, __nv_bfloat16);
+    else if (epilogue == GV_RELU2 && out_dtype == DT_BF16) rc = EL_GV(__nv_bfloat16, GV_RELU2, __nv_bfloat16);
     else EL_REFUSE(false, "gemv: unsupported epilogue %d with output dtype %d", epilogue, out_dtype);
   } else if (dtype == DT_F32) {
     EL_REFUSE(out_dtype == DT_F32, "gemv: float32 activations give float32 outputs");
     if (epilogue == GV_STORE) rc = EL_GV(float, GV_STORE, float);
     else if (epilogue == GV_RESIDUAL) rc = EL_GV(float, GV_RESIDUAL, float);
     else if (epilogue == GV_SWIGLU) rc = EL_GV(float, GV_SWIGLU, float);
+    else if (epilogue == GV_RELU2) rc = EL_GV(float, GV_RELU2, float);
     else EL_REFUSE(false, "gemv: unknown epilogue %d", epilogue);
   } else {
     EL_REFUSE(false, "gemv: unknown dtype code %d", dtype);

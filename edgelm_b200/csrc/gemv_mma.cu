@@ -15,7 +15,7 @@
 //   * the activations of all rows sit in shared memory (pitch chosen so that the fragment reads
 //     hit distinct banks), optionally produced here as RMSNorm(x) from the float32 residual
 //     stream, rounded to bfloat16 as the stand-alone norm kernel rounds;
-//   * epilogues: store (bfloat16 or float32), += residual (float32), SwiGLU of two weights.
+//   * epilogues: store (bfloat16 or float32), += residual (float32), SwiGLU of two weights, squared ReLU (bfloat16).
 // K must be a multiple of 8 with 16-byte aligned rows; M <= 16.  Launched as a programmatic dependent
 // launch: the first weight loads are issued before the wait for the previous kernel.
 // A launch can be told the weights that the step reads next (`edgelm_gemv_mma_prefetch_next`): its blocks then ask
@@ -25,7 +25,7 @@
 
 namespace edgelm {
 
-enum : int { GM_STORE = 0, GM_RESIDUAL = 1, GM_SWIGLU = 2 };
+enum : int { GM_STORE = 0, GM_RESIDUAL = 1, GM_SWIGLU = 2, GM_RELU2 = 4 };
 constexpr int GM_MAX_WARPS = 16;
 constexpr int GM_COLS = 16;  // output columns per block
 constexpr int GM_K_CHUNK = 4096;  // columns of the activations in shared memory at a time
@@ -327,6 +327,7 @@ gemv_mma_kernel(const __nv_bfloat16* __restrict__ act, int lda, const float* __r
         if (EPI == GM_STORE) out[idx] = from_f32<TOut>(s[0][j]);
         if (EPI == GM_RESIDUAL) out[idx] = from_f32<TOut>(res_ahead[t][j] + s[0][j]);
         if (EPI == GM_SWIGLU) out[idx] = from_f32<TOut>(gm_silu(s[0][j]) * s[NW - 1][j]);
+        if (EPI == GM_RELU2) out[idx] = from_f32<TOut>(fmaxf(s[0][j], 0.f) * fmaxf(s[0][j], 0.f));
       }
     }
   }
@@ -502,6 +503,7 @@ gemv_mma_walk_kernel(const __nv_bfloat16* __restrict__ act, int lda, const __nv_
           const size_t idx = (size_t)m * ldo + n;
           if (EPI == GM_STORE) out[idx] = from_f32<TOut>(s[0][j]);
           if (EPI == GM_SWIGLU) out[idx] = from_f32<TOut>(gm_silu(s[0][j]) * s[NW - 1][j]);
+          if (EPI == GM_RELU2) out[idx] = from_f32<TOut>(fmaxf(s[0][j], 0.f) * fmaxf(s[0][j], 0.f));
         }
       }
     }
@@ -655,6 +657,7 @@ extern "C" int edgelm_gemv_mma(const void* act, int lda, const float* norm_w, fl
   else if (epilogue == GM_STORE && out_dtype == DT_F32) EL_GM(GM_STORE, float);
   else if (epilogue == GM_RESIDUAL) EL_GM(GM_RESIDUAL, float);
   else if (epilogue == GM_SWIGLU && out_dtype == DT_BF16) EL_GM(GM_SWIGLU, __nv_bfloat16);
+  else if (epilogue == GM_RELU2 && out_dtype == DT_BF16) EL_GM(GM_RELU2, __nv_bfloat16);
   else EL_REFUSE(false, "gemv_mma: unsupported epilogue %d with output dtype %d", epilogue, out_dtype);
 #undef EL_GM
   g_next[0] = g_next[1] = NextWeights{nullptr, 0};

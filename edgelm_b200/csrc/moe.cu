@@ -2,9 +2,9 @@
 //
 //   route     logits z = Wr h + br in float32 (a block a token); the `top` largest (first maximum on ties), and their
 //             weights: the softmax over the chosen logits only.
-//   route_scored   another router on the same logits: scores s = softmax(z) over all experts; the choice looks at s + a
-//             correction per expert, optionally only inside the `keep` groups of neighbouring experts whose best corrected
-//             score is largest; the weights are the chosen experts' s over their sum, times a constant.  The last experts may
+//   route_scored   another router on the same logits: scores s = softmax(z) over all experts, or each expert's sigmoid(z); the
+//             choice looks at s + a correction per expert, optionally only inside the `keep` groups of neighbouring experts whose
+//             best corrected score is largest; the weights are the chosen experts' s, as they are or over their sum, times a constant.  The last experts may
 //             be "identity experts" without weights (they give back their input): their pairs get no row, and `combine`
 //             adds the token's own input for them.  Extra router rows after the experts give per-token gates (sigmoid).
 //   plan      the (token, choice) pairs are grouped by expert: rows of a padded layout in which every expert's rows
@@ -12,8 +12,9 @@
 //             row_pair[row] = pair (token * top + choice) or -1; pair_row[pair] = its row; tile_expert[tile] = expert or -1.
 //   products  mid[row] = silu(Wg_e h) * (Wu_e h) for the row's token; y[row] = Wd_e mid[row] (float32): on the CUDA
 //             cores here (float32 models, sizes the tensor-core kernel does not take), or by the grouped tcgen05 product
-//             over rows gathered by `gather_rows` (row tiles of 128).
-//   combine   x[t] += sum_k weight[t][k] * y[pair_row[t * top + k]], in the order of k.
+//             over rows gathered by `gather_rows` (row tiles of 128).  A pair's weight may act on the expert's input instead of its
+//             output: both products are linear in the input, so it multiplies their float32 sums before the unit.
+//   combine   x[t] += sum_k weight[t][k] * y[pair_row[t * top + k]], in the order of k (weight 1 where it acted on the input).
 // Every row is computed by itself, so a token's result does not depend on what else is in the step.
 #include "common.cuh"
 
@@ -82,13 +83,15 @@ moe_route_kernel(const TH* __restrict__ h, const float* __restrict__ wr, const f
   }
 }
 
+enum : int { SCORE_SOFTMAX = 0, SCORE_SIGMOID = 1 };
+
 // The scored router (see the head of this file).  E experts in all (the last ones may be identity experts: nothing here
 // treats them differently), `n_extra` more router rows whose sigmoid goes to extra[t][.].  Ties: the first of equal scores.
 template <typename TH>
 __global__ void __launch_bounds__(128)
 moe_route_scored_kernel(const TH* __restrict__ h, const float* __restrict__ wr, const float* __restrict__ correction,
                         int32_t* __restrict__ idx, float* __restrict__ wts, float* __restrict__ extra, int D, int E, int n_extra, int top,
-                        int groups, int keep, float scale) {
+                        int groups, int keep, float scale, int score, int renormalize) {
   pdl_launch_dependents();
   pdl_wait();
   extern __shared__ float mr_smem[];         // [E + n_extra] logits, [E] choice scores, [groups] group scores, then [4][8] partial sums
@@ -98,7 +101,13 @@ moe_route_scored_kernel(const TH* __restrict__ h, const float* __restrict__ wr, 
   const int t = blockIdx.x;
   moe_logits(h + (size_t)t * D, wr, (const float*)nullptr, z, gs + groups, D, E + n_extra);
   if (threadIdx.x < n_extra) extra[(size_t)t * n_extra + threadIdx.x] = 1.0f / (1.0f + expf(-z[E + threadIdx.x]));
-  if (threadIdx.x == 0) {
+  // z <- the scores, c <- what the choice looks at
+  if (score == SCORE_SIGMOID) {
+    for (int e = threadIdx.x; e < E; e += blockDim.x) {
+      z[e] = 1.0f / (1.0f + expf(-z[e]));
+      c[e] = z[e] + (correction ? correction[e] : 0.f);
+    }
+  } else if (threadIdx.x == 0) {
     float zmax = -INFINITY, sum = 0.f;
     for (int e = 0; e < E; ++e) zmax = fmaxf(zmax, z[e]);
     for (int e = 0; e < E; ++e) {
@@ -107,10 +116,15 @@ moe_route_scored_kernel(const TH* __restrict__ h, const float* __restrict__ wr, 
     }
     const float inv = 1.0f / sum;
     for (int e = 0; e < E; ++e) {
-      z[e] *= inv;                                  // the score
-      c[e] = z[e] + (correction ? correction[e] : 0.f);   // what the choice looks at
+      z[e] *= inv;
+      c[e] = z[e] + (correction ? correction[e] : 0.f);
     }
-    if (groups > 1) {
+  }
+  __syncthreads();
+  if (threadIdx.x >= 32) return;             // one warp chooses
+  const int lane = threadIdx.x;
+  if (groups > 1) {
+    if (lane == 0) {
       const int size = E / groups;
       for (int g = 0; g < groups; ++g) {
         float b = -INFINITY;
@@ -125,28 +139,37 @@ moe_route_scored_kernel(const TH* __restrict__ h, const float* __restrict__ wr, 
           for (int e = g * size; e < (g + 1) * size; ++e) c[e] = -INFINITY;
       }
     }
-    float picked = 0.f;
-    for (int k = 0; k < top; ++k) {
-      int best = -1;
-      float bc = -INFINITY;
-      for (int e = 0; e < E; ++e)
-        if (c[e] > bc) { bc = c[e]; best = e; }
-      if (best < 0)         // fewer allowed experts than `top`: the left-out ones follow in the order of their numbers
-        for (int e = 0; e < E && best < 0; ++e)
-          if (c[e] == -INFINITY) best = e;
-      if (best < 0) {       // (nothing left at all: NaN scores)
-        idx[(size_t)t * top + k] = -1;
-        wts[(size_t)t * top + k] = 0.f;
-        continue;
-      }
-      idx[(size_t)t * top + k] = best;
-      wts[(size_t)t * top + k] = z[best];
-      picked += z[best];
-      c[best] = NAN;        // taken (compares false with everything; a left-out expert stays at minus infinity)
-    }
-    const float norm = scale / (picked + 1e-20f);
-    for (int k = 0; k < top; ++k) wts[(size_t)t * top + k] *= norm;
+    __syncwarp();
   }
+  float picked = 0.f;
+  for (int k = 0; k < top; ++k) {
+    // lane l looks at the experts l, l + 32, ...: the largest (the first of equal ones), and the first left-out one
+    int best = -1, left_out = E;
+    float bc = -INFINITY;
+    for (int e = lane; e < E; e += 32) {
+      if (c[e] > bc) { bc = c[e]; best = e; }
+      else if (c[e] == -INFINITY) left_out = min(left_out, e);
+    }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+      const float oc = __shfl_xor_sync(0xffffffffu, bc, o);
+      const int ob = __shfl_xor_sync(0xffffffffu, best, o);
+      left_out = min(left_out, __shfl_xor_sync(0xffffffffu, left_out, o));
+      if (ob >= 0 && (best < 0 || oc > bc || (oc == bc && ob < best))) { bc = oc; best = ob; }
+    }
+    if (best < 0 && left_out < E) best = left_out;     // fewer allowed experts than `top`: the left-out ones follow in the order of their numbers
+    const float s = best >= 0 ? z[best] : 0.f;         // (best < 0: nothing left at all, NaN scores)
+    picked += s;
+    if (lane == 0) {
+      idx[(size_t)t * top + k] = best;
+      wts[(size_t)t * top + k] = s;
+      if (best >= 0) c[best] = NAN;          // taken (compares false with everything; a left-out expert stays at minus infinity)
+    }
+    __syncwarp();
+  }
+  const float norm = renormalize ? scale / (picked + 1e-20f) : scale;
+  if (lane == 0 && norm != 1.0f)
+    for (int k = 0; k < top; ++k) wts[(size_t)t * top + k] *= norm;
 }
 
 // One block.  counts -> padded offsets -> rows.  The order of an expert's rows depends on the order in which the threads
@@ -204,6 +227,7 @@ __global__ void moe_gather_rows_kernel(const T* __restrict__ h, T* __restrict__ 
 
 // The products on the CUDA cores (float32 sums): tiles of 32 rows x 64 columns, K in steps of 32 through shared memory.
 //   GATED: a[row] = h[row_pair[row] / top]; out[row][n] = silu(a . wg_e[n]) * (a . wu_e[n])          (mid, type T)
+//          (`in_weight`: both sums times in_weight[row_pair[row]] first, the pair's weight on the expert's input)
 //   else:  a[row] = mid[row];               y[row][n] = a . w_e[n]                                    (float32)
 constexpr int MG_TM = 32, MG_TN = 64, MG_KC = 32;
 
@@ -211,7 +235,7 @@ template <typename T, bool GATED>
 __global__ void __launch_bounds__(256)
 moe_gemm_kernel(const T* __restrict__ a, int lda, const T* __restrict__ w, const T* __restrict__ w2, void* __restrict__ out, int ldo,
                 const int32_t* __restrict__ row_pair, const int32_t* __restrict__ tile_expert, int top, int K, int N, float glu_limit,
-                float glu_alpha, float glu_shift) {
+                float glu_alpha, float glu_shift, const float* __restrict__ in_weight) {
   pdl_launch_dependents();
   pdl_wait();
   const int e = tile_expert[blockIdx.x];
@@ -263,13 +287,14 @@ moe_gemm_kernel(const T* __restrict__ a, int lda, const T* __restrict__ w, const
   for (int i = 0; i < 2; ++i) {
     const int r = ty * 2 + i, p = pair_of[r];
     if (p < 0) continue;
+    const float iw = GATED && in_weight ? in_weight[p] : 1.0f;
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       const int n = n0 + tx + 16 * j;
       if (n >= N) continue;
       if (GATED) {
         // the gated unit: g sigmoid(alpha g) (v + shift), both branches clamped when there is a limit (none, 1, 0: SwiGLU)
-        float z = acc[i][j], v = acc2[i][j];
+        float z = acc[i][j] * iw, v = acc2[i][j] * iw;
         if (glu_limit > 0.f) {
           z = fminf(z, glu_limit);
           v = fminf(fmaxf(v, -glu_limit), glu_limit);
@@ -282,7 +307,7 @@ moe_gemm_kernel(const T* __restrict__ a, int lda, const T* __restrict__ w, const
   }
 }
 
-// x[t][:] += sum_k wts[t][k] * y[pair_row[t * top + k]][:]  (+ gate[t] * shared[t][:])
+// x[t][:] += sum_k wts[t][k] * y[pair_row[t * top + k]][:]  (+ gate[t] * shared[t][:]); wts null: every weight is 1
 // A pair without a row whose expert number is at least `n_real` is an identity expert's: its output is the token's own input
 // h[t] (in the type the experts read it in).
 template <typename TH>
@@ -296,8 +321,9 @@ __global__ void moe_combine_kernel(float* __restrict__ x, const float* __restric
     float acc = 0.f;
     for (int k = 0; k < top; ++k) {
       const int r = pair_row[(size_t)t * top + k];
-      if (r >= 0) acc = fmaf(wts[(size_t)t * top + k], y[(size_t)r * ldy + i], acc);
-      else if (idx && idx[(size_t)t * top + k] >= n_real) acc = fmaf(wts[(size_t)t * top + k], to_f32(h[(size_t)t * D + i]), acc);
+      const float w = wts ? wts[(size_t)t * top + k] : 1.0f;
+      if (r >= 0) acc = fmaf(w, y[(size_t)r * ldy + i], acc);
+      else if (idx && idx[(size_t)t * top + k] >= n_real) acc = fmaf(w, to_f32(h[(size_t)t * D + i]), acc);
     }
     if (shared) acc = fmaf(gate ? gate[t] : 1.0f, shared[(size_t)t * D + i], acc);
     x[(size_t)t * D + i] += acc;
@@ -326,16 +352,17 @@ extern "C" int edgelm_moe_route(const void* h, int dtype, const float* wr, const
 
 extern "C" int edgelm_moe_route_scored(const void* h, int dtype, const float* wr, const float* correction, int32_t* idx, float* wts,
                                        float* extra, int n_tokens, int D, int E, int n_extra, int top, int groups, int keep, float scale,
-                                       cudaStream_t stream) {
+                                       int score, int renormalize, cudaStream_t stream) {
   if (n_tokens == 0) return 0;
   EL_REFUSE(n_tokens > 0 && D > 0 && E >= 1 && E <= MOE_MAX_EXPERTS && top >= 1 && top <= E, "moe_route_scored: %d experts, %d chosen", E, top);
   EL_REFUSE(groups >= 1 && E % groups == 0 && keep >= 1 && keep <= groups, "moe_route_scored: %d experts in %d groups, %d kept", E, groups, keep);
   EL_REFUSE(n_extra >= 0 && n_extra <= 32 && (n_extra == 0 || extra != nullptr), "moe_route_scored: %d extra rows (up to 32)", n_extra);
+  EL_REFUSE(score == SCORE_SOFTMAX || score == SCORE_SIGMOID, "moe_route_scored: unknown score %d", score);
   const dim3 grid(n_tokens), block(128);
   const size_t smem = (size_t)(2 * E + n_extra + groups + 32) * sizeof(float);
   const int bit = pdl_bit_for_tokens(n_tokens);
-  if (dtype == DT_F32) launch_pdl(bit, moe_route_scored_kernel<float>, grid, block, smem, stream, (const float*)h, wr, correction, idx, wts, extra, D, E, n_extra, top, groups, keep, scale);
-  else if (dtype == DT_BF16) launch_pdl(bit, moe_route_scored_kernel<__nv_bfloat16>, grid, block, smem, stream, (const __nv_bfloat16*)h, wr, correction, idx, wts, extra, D, E, n_extra, top, groups, keep, scale);
+  if (dtype == DT_F32) launch_pdl(bit, moe_route_scored_kernel<float>, grid, block, smem, stream, (const float*)h, wr, correction, idx, wts, extra, D, E, n_extra, top, groups, keep, scale, score, renormalize);
+  else if (dtype == DT_BF16) launch_pdl(bit, moe_route_scored_kernel<__nv_bfloat16>, grid, block, smem, stream, (const __nv_bfloat16*)h, wr, correction, idx, wts, extra, D, E, n_extra, top, groups, keep, scale, score, renormalize);
   else EL_REFUSE(false, "moe_route_scored: unknown dtype code %d", dtype);
   EL_LAUNCH_CHECK("moe_route_scored");
   return 0;
@@ -352,15 +379,16 @@ extern "C" int edgelm_moe_plan(const int32_t* idx, int n_pairs, int E, int tile_
 }
 
 // gated != 0: the gate and up products with the activation; a = the tokens' rows [tokens][K]; out = mid [rows][N] in `dtype`.
+// `in_weight` (or null): a float per (token, choice) pair that multiplies the expert's input.
 // gated == 0: the down product; a = mid [rows][K]; out = y [rows][N] float32.
 extern "C" int edgelm_moe_gemm(const void* a, int lda, const void* w, const void* w2, void* out, int ldo, const int32_t* row_pair,
                                const int32_t* tile_expert, int max_tiles, int top, int K, int N, int dtype, int gated, float glu_limit, float glu_alpha,
-                               float glu_shift, cudaStream_t stream) {
+                               float glu_shift, const float* in_weight, cudaStream_t stream) {
   if (max_tiles == 0) return 0;
   EL_REFUSE(max_tiles > 0 && K > 0 && N > 0 && top >= 1, "moe_gemm: bad sizes");
   const dim3 grid(max_tiles, (N + MG_TN - 1) / MG_TN), block(256);
   const int bit = pdl_bit_for_tokens(max_tiles);
-#define EL_MG(T, GATED) launch_pdl(bit, moe_gemm_kernel<T, GATED>, grid, block, (size_t)0, stream, (const T*)a, lda, (const T*)w, (const T*)w2, out, ldo, row_pair, tile_expert, top, K, N, glu_limit, glu_alpha, glu_shift)
+#define EL_MG(T, GATED) launch_pdl(bit, moe_gemm_kernel<T, GATED>, grid, block, (size_t)0, stream, (const T*)a, lda, (const T*)w, (const T*)w2, out, ldo, row_pair, tile_expert, top, K, N, glu_limit, glu_alpha, glu_shift, in_weight)
   if (dtype == DT_F32 && gated) EL_MG(float, true);
   else if (dtype == DT_F32) EL_MG(float, false);
   else if (dtype == DT_BF16 && gated) EL_MG(__nv_bfloat16, true);

@@ -15,7 +15,7 @@ import torch
 from . import build as _build
 
 F32, BF16 = 0, 1
-EPI_STORE, EPI_RESIDUAL, EPI_SWIGLU = 0, 1, 2
+EPI_STORE, EPI_RESIDUAL, EPI_SWIGLU, EPI_RELU2 = 0, 1, 2, 4     # (3 is the rotation epilogue, which has an entry of its own)
 PAGE = 64  # tokens per cache page, as in common.cuh
 
 ERR_BITS = {1: "a token id outside the vocabulary", 2: "a position beyond the position table",
@@ -464,6 +464,11 @@ def _f32(t, name):
     _need(t.dtype == torch.float32 and t.is_cuda and t.is_contiguous(), f"{name} must be a contiguous float32 CUDA tensor")
 
 
+def _f32_rows(t, name):
+    """Float32 rows of any pitch (a slice of a wider product's columns, say)."""
+    _need(t.dtype == torch.float32 and t.is_cuda and t.dim() == 2 and t.stride(1) == 1, f"{name} must be float32 rows on the device")
+
+
 def shift_mix(inp, state, mu, out, tok_seq, seq_tok0, seq_slot, move_state=False):
     """out[m, t] = a + (prev - a) * mu[m] with a = inp[t] and prev the row before it, or the sequence's state row for
     the first token that the sequence brings to this step.  inp [T, D] float32 or bfloat16; mu [M, D]; out [M, T, D].
@@ -663,9 +668,10 @@ def _masked_cache_check(kcache, vcache, nkv, dk, dv, what):
 
 
 def rotate_append(qkv, bias, q_out, tok_pos, tok_seq, page_table, kcache, vcache, nh, nkv, dk, dv, rot, interleaved, freq, err,
-                  maps=1, q_norm=None, k_norm=None, eps=0.0, conv_w=None, conv_state=None, seq_tok0=None, seq_slot=None, n_seqs=0):
+                  maps=1, q_norm=None, k_norm=None, eps=0.0, conv_w=None, conv_state=None, seq_tok0=None, seq_slot=None, n_seqs=0, rot_mult=1.0):
     """qkv [T, nh dk + nkv dk + nkv dv] float32 (+ bias): the first `rot` dimensions of every query and key head are rotated
-    by position * freq (float64 frequencies; pairs (2i, 2i + 1) if `interleaved`, else (i, i + rot/2)); queries go to q_out
+    by position * freq (float64 frequencies; pairs (2i, 2i + 1) if `interleaved`, else (i, i + rot/2); sine and cosine times `rot_mult`);
+    queries go to q_out
     [T, nh dk] float32, keys and values to their places in the cache pages.  `maps` > 1: a head of dk dimensions is `maps`
     runs of dk / maps side by side, each rotated (its first `rot` dimensions) by itself.  `q_norm` / `k_norm` (float32
     [dk / maps]): every run is first divided by its root mean square (`eps` inside the root) and multiplied by the weight.
@@ -699,19 +705,19 @@ def rotate_append(qkv, bias, q_out, tok_pos, tok_seq, page_table, kcache, vcache
                                       kcache.shape[0], _p(kcache), _p(vcache), _dt(kcache), T, nh, nkv, dk, dv, int(rot),
                                       1 if interleaved else 0, _p(freq), _p(err), int(maps), _p(q_norm), _p(k_norm), ctypes.c_float(eps),
                                       qkv.stride(0), _p(conv_w), int(taps), _p(conv_state if taps > 1 else None), _p(seq_tok0), _p(seq_slot),
-                                      1 if single else 0, _stream()))
+                                      1 if single else 0, ctypes.c_float(rot_mult), _stream()))
     if conv_w is not None and taps > 1 and not single:
         _check(lib().edgelm_conv_tail_update(_p(qkv), qkv.stride(0), 0, _p(conv_state), _p(seq_tok0), _p(seq_slot), int(n_seqs), qkv.shape[1], int(taps),
                                              _p(bias), _stream()))
 
 
 def latent_prepare(u, kv_off, has_kv, q_out, q_pitch, q_off, copy_q, norm_w, eps, tok_pos, tok_seq, page_table, kcache, nh, d, rd, r, freq, err,
-                   row_out=None):
+                   row_out=None, interleaved=False, rot_mult=1.0):
     """u [T, *] float32: nh query heads of [d | rd] from column 0 and, with `has_kv`, the latent's row [r | rd] from column
-    `kv_off`.  The rotated part of every query head (pairs (i, i + rd/2)) goes to q_out[t, h * q_pitch + q_off :], with
+    `kv_off`.  The rotated part of every query head (pairs and `rot_mult` as in `rotate_append`) goes to q_out[t, h * q_pitch + q_off :], with
     `copy_q` the unrotated part to q_out[t, h * q_pitch :]; the latent, RMS-normed with `norm_w`, and the rotated shared key
     part become the token's cache row [r + rd], and row t of `row_out` [T, r + rd] (optional, the cache's type)."""
-    _f32(u, "u"); _f32(q_out, "q_out")
+    _f32_rows(u, "u"); _f32(q_out, "q_out")
     T = u.shape[0]
     _need(q_out.shape == (T, nh * q_pitch), "latent_prepare: q_out shape")
     _need(rd == 0 or (freq is not None and freq.dtype == torch.float64 and freq.numel() == rd // 2 and freq.is_contiguous()), "latent_prepare: frequencies")
@@ -727,7 +733,7 @@ def latent_prepare(u, kv_off, has_kv, q_out, q_pitch, q_off, copy_q, norm_w, eps
                                        _p(norm_w) if has_kv else _p(None), ctypes.c_float(eps), _p(tok_pos), _p(tok_seq),
                                        _p(page_table) if has_kv else _p(None), page_table.stride(0) if has_kv else 0, kcache.shape[0] if has_kv else 0,
                                        _p(kcache) if has_kv else _p(None), _p(row_out) if has_kv else _p(None), _dt(kcache) if has_kv else F32,
-                                       T, nh, d, rd, r, _p(freq), _p(err), _stream()))
+                                       T, nh, d, rd, r, _p(freq), _p(err), 1 if interleaved else 0, ctypes.c_float(rot_mult), _stream()))
 
 
 def latent_expand_keys(kn, rows, kx, nh, d, rd, r):
@@ -741,7 +747,7 @@ def latent_expand_keys(kn, rows, kx, nh, d, rd, r):
 def head_matmul(a, a_head_stride, w, out, out_head_stride):
     """out[t, h * out_head_stride + n] = sum_k a[t, h * a_head_stride + k] * w[h, n, k]: one small product per head.
     a float32 rows; w [heads, N, K] float32 or bfloat16; out float32 or the weights' type."""
-    _f32(a, "a")
+    _f32_rows(a, "a")
     _need(w.dim() == 3 and w.is_contiguous() and out.stride(1) == 1 and a.stride(1) == 1, "head_matmul: layout")
     H, N, K = w.shape
     _need((H - 1) * a_head_stride + K <= a.shape[1] and (H - 1) * out_head_stride + N <= out.shape[1] and out.shape[0] == a.shape[0], "head_matmul: shapes")
@@ -893,12 +899,16 @@ def moe_route(h, wr, br, idx, wts, top):
     _check(lib().edgelm_moe_route(_p(h), _dt(h), _p(wr), _p(br), _p(idx), _p(wts), T, D, E, int(top), _stream()))
 
 
-def moe_route_scored(h, wr, correction, idx, wts, top, n_experts, groups=1, keep=1, scale=1.0, extra=None):
-    """The router that scores every expert: s = softmax(wr[:n_experts] h) over all experts (float32); the `top` experts with the
+ROUTER_SCORES = {"softmax": 0, "sigmoid": 1}
+
+
+def moe_route_scored(h, wr, correction, idx, wts, top, n_experts, groups=1, keep=1, scale=1.0, extra=None, score="softmax", renormalize=True):
+    """The router that scores every expert: s = softmax(wr[:n_experts] h) over all experts, or sigmoid(wr[e] h) expert by expert
+    (float32); the `top` experts with the
     largest s + correction are chosen (first of equal ones), with `groups` > 1 only among the `keep` groups of neighbouring
     experts whose best corrected score is largest (the others count as minus infinity: when the kept groups hold fewer than `top`
-    experts, the left-out ones follow in the order of their numbers); wts = s of the chosen over their sum (+ 1e-20), times
-    `scale`.  Rows of `wr` after the first `n_experts` give `extra` [T, rows] = sigmoid(row . h).  idx of a choice that could not
+    experts, the left-out ones follow in the order of their numbers); wts = s of the chosen over their sum (+ 1e-20; not
+    `renormalize`: s as it is), times `scale`.  Rows of `wr` after the first `n_experts` give `extra` [T, rows] = sigmoid(row . h).  idx of a choice that could not
     be made (scores that are not numbers): -1."""
     _f32(wr, "router weight"); _f32(wts, "wts"); _i32(idx, "idx")
     T, D = h.shape
@@ -907,7 +917,7 @@ def moe_route_scored(h, wr, correction, idx, wts, top, n_experts, groups=1, keep
     _need(correction is None or (correction.dtype == torch.float32 and correction.is_contiguous() and correction.numel() == n_experts), "moe_route_scored: correction")
     _need((n_extra == 0) == (extra is None) and (extra is None or (extra.dtype == torch.float32 and extra.is_contiguous() and extra.shape == (T, n_extra))), "moe_route_scored: extra rows")
     _check(lib().edgelm_moe_route_scored(_p(h), _dt(h), _p(wr), _p(correction), _p(idx), _p(wts), _p(extra), T, D, int(n_experts), int(n_extra), int(top),
-                                         int(groups), int(keep), ctypes.c_float(scale), _stream()))
+                                         int(groups), int(keep), ctypes.c_float(scale), ROUTER_SCORES[score], 1 if renormalize else 0, _stream()))
 
 
 def moe_plan(idx, n_experts, tile_rows, row_pair, pair_row, tile_expert):
@@ -926,19 +936,26 @@ def moe_gather_rows(h, a, row_pair, top):
     _check(lib().edgelm_moe_gather_rows(_p(h), _p(a), _p(row_pair), row_pair.numel(), int(top), h.shape[1], _dt(h), _stream()))
 
 
+def _pair_weights(w, what):
+    _need(w is None or (w.dtype == torch.float32 and w.is_cuda and w.is_contiguous()), f"{what}: the pairs' weights")
+    return w
+
+
 GLU_SWIGLU = (0.0, 1.0, 0.0)     # (limit, alpha, shift) of the gated unit g sigmoid(alpha g) (v + shift); limit 0: no clamps
 
 
-def moe_gate_up(h, w_gate, w_up, mid, row_pair, tile_expert, top, glu=GLU_SWIGLU):
+def moe_gate_up(h, w_gate, w_up, mid, row_pair, tile_expert, top, glu=GLU_SWIGLU, in_weight=None):
     """mid[row] = unit(w_gate[e] h[t], w_up[e] h[t]) for every row of the plan (t = row_pair[row] // top, e the row's tile's
     expert), on the CUDA cores.  The unit is silu(g) * v, or with `glu` (limit, alpha, shift) g sigmoid(alpha g) (v + shift) with
-    g = min(g, limit) and v = clamp(v, -limit, limit) when limit > 0."""
+    g = min(g, limit) and v = clamp(v, -limit, limit) when limit > 0.  `in_weight` (float32, one per pair): multiplies the
+    pair's input h[t] (the two products' float32 sums, which are linear in it)."""
     E, N, K = w_gate.shape
     _need(h.dtype == w_gate.dtype == w_up.dtype == mid.dtype and h.is_contiguous() and w_gate.is_contiguous() and w_up.is_contiguous() and mid.is_contiguous(), "moe_gate_up: layout")
     _need(h.shape[1] == K and w_up.shape == w_gate.shape and mid.shape == (row_pair.numel(), N), "moe_gate_up: shapes")
     _need(row_pair.numel() == tile_expert.numel() * moe_tile_rows(), "moe_gate_up: the plan's row tile is not this kernel's")
     _check(lib().edgelm_moe_gemm(_p(h), h.stride(0), _p(w_gate), _p(w_up), _p(mid), mid.stride(0), _p(row_pair), _p(tile_expert),
-                                 tile_expert.numel(), int(top), K, N, _dt(h), 1, ctypes.c_float(glu[0]), ctypes.c_float(glu[1]), ctypes.c_float(glu[2]), _stream()))
+                                 tile_expert.numel(), int(top), K, N, _dt(h), 1, ctypes.c_float(glu[0]), ctypes.c_float(glu[1]), ctypes.c_float(glu[2]),
+                                 _p(_pair_weights(in_weight, "moe_gate_up")), _stream()))
 
 
 def moe_down(mid, w_down, y, row_pair, tile_expert, top):
@@ -948,7 +965,7 @@ def moe_down(mid, w_down, y, row_pair, tile_expert, top):
     _need(mid.dtype == w_down.dtype and mid.is_contiguous() and w_down.is_contiguous() and mid.shape == (row_pair.numel(), K) and y.shape == (row_pair.numel(), N), "moe_down: shapes")
     _need(row_pair.numel() == tile_expert.numel() * moe_tile_rows(), "moe_down: the plan's row tile is not this kernel's")
     _check(lib().edgelm_moe_gemm(_p(mid), mid.stride(0), _p(w_down), _p(None), _p(y), y.stride(0), _p(row_pair), _p(tile_expert),
-                                 tile_expert.numel(), int(top), K, N, _dt(mid), 0, ctypes.c_float(0.0), ctypes.c_float(1.0), ctypes.c_float(0.0), _stream()))
+                                 tile_expert.numel(), int(top), K, N, _dt(mid), 0, ctypes.c_float(0.0), ctypes.c_float(1.0), ctypes.c_float(0.0), _p(None), _stream()))
 
 
 def gemm_tc_grouped_takes(a, w, w2=None):
@@ -958,27 +975,35 @@ def gemm_tc_grouped_takes(a, w, w2=None):
     return bool(lib().edgelm_gemm_tc_takes(_p(a), a.stride(0), _p(w), _p(w2), a.shape[1]))
 
 
-def gemm_tc_grouped(a, w, out, tile_group, err, epilogue=EPI_STORE, w2=None, glu=GLU_SWIGLU):
+def gemm_tc_grouped(a, w, out, tile_group, err, epilogue=EPI_STORE, w2=None, glu=GLU_SWIGLU, row_pair=None, in_weight=None):
     """out[row] = a[row] @ w[g].T (+ epilogue) with g = tile_group[row // 128] (negative: a tile without rows): a [M, K]
     bfloat16 with M a multiple of 128, w (and w2 for the gated unit) [groups, N, K] bfloat16, out [M, N] float32 or bfloat16.
-    `glu`: the gated unit's form, as in `moe_gate_up`."""
+    `glu`: the gated unit's form, as in `moe_gate_up`; `in_weight` (one per pair, with `row_pair` [M]): the pairs' weights on the input."""
     _i32(tile_group, "tile_group")
     G, N, K = w.shape
     M = a.shape[0]
     _need(a.shape == (M, K) and out.shape == (M, N) and out.stride(1) == 1 and tile_group.numel() * 128 == M, "gemm_tc_grouped: shapes")
     _need(w2 is None or (w2.shape == w.shape and w2.is_contiguous() and w2.dtype == w.dtype), "gemm_tc_grouped: second weight")
+    if in_weight is not None:
+        _i32(row_pair, "row_pair")
+        _need(row_pair.numel() == M and epilogue == EPI_SWIGLU, "gemm_tc_grouped: weights on the input need the rows' pairs and the gated unit")
     _check(lib().edgelm_gemm_tc_grouped(_p(a), a.stride(0), _p(w), _p(w2), _p(out), out.stride(0), M, N, K, G, _p(tile_group), _dt(out), int(epilogue),
-                                        ctypes.c_float(glu[0]), ctypes.c_float(glu[1]), ctypes.c_float(glu[2]), _p(err), _stream()))
+                                        ctypes.c_float(glu[0]), ctypes.c_float(glu[1]), ctypes.c_float(glu[2]), _p(row_pair if in_weight is not None else None),
+                                        _p(_pair_weights(in_weight, "gemm_tc_grouped")), _p(err), _stream()))
 
 
-def moe_combine(x, y, wts, pair_row, idx=None, n_real=0, h=None, shared=None, gate=None):
-    """x[t] += sum_k wts[t, k] * y[pair_row[t * top + k]].  With `idx` [T, top], `n_real` and `h` [T, D]: a pair whose expert
+def moe_combine(x, y, wts, pair_row, idx=None, n_real=0, h=None, shared=None, gate=None, top=None):
+    """x[t] += sum_k wts[t, k] * y[pair_row[t * top + k]] (`wts` None with `top` given: every weight is 1).  With `idx` [T, top], `n_real` and `h` [T, D]: a pair whose expert
     number is at least `n_real` belongs to an identity expert, whose output is the token's input h[t].  With `shared`
     [T, D] float32 (and `gate` [T] float32, else 1): x[t] += gate[t] * shared[t] as well."""
-    _f32(x, "x"); _f32(y, "y"); _f32(wts, "wts"); _i32(pair_row, "pair_row")
-    T, top = wts.shape
-    D = x.shape[1]
-    _need(x.shape[0] == T and y.shape[1] == D and pair_row.numel() == T * top, "moe_combine: shapes")
+    _f32(x, "x"); _f32(y, "y"); _i32(pair_row, "pair_row")
+    T, D = x.shape
+    if wts is not None:
+        _f32(wts, "wts")
+        _need(top is None or top == wts.shape[1], "moe_combine: choices a token")
+        top = wts.shape[1]
+    _need(top is not None and (wts is None or wts.shape[0] == T), "moe_combine: choices a token")
+    _need(y.shape[1] == D and pair_row.numel() == T * top, "moe_combine: shapes")
     if idx is not None:
         _i32(idx, "idx")
         _need(idx.numel() == T * top and h is not None and h.is_contiguous() and h.shape == (T, D), "moe_combine: identity experts need the tokens' inputs")

@@ -14,7 +14,7 @@ import torch
 
 from ..csrc import ops
 
-EPI_STORE, EPI_RESIDUAL, EPI_SWIGLU = ops.EPI_STORE, ops.EPI_RESIDUAL, ops.EPI_SWIGLU
+EPI_STORE, EPI_RESIDUAL, EPI_SWIGLU, EPI_RELU2 = ops.EPI_STORE, ops.EPI_RESIDUAL, ops.EPI_SWIGLU, ops.EPI_RELU2
 
 FEW_ROWS = 16  # up to here one pass over the weights with all rows in shared memory is bandwidth-bound already
 MMA_MIN_ROWS = 1        # rows from which the tensor-core few-rows kernel is used (measured: never slower)

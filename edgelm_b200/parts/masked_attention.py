@@ -4,7 +4,7 @@ q, k, v are projections of the mixer's input (one matrix product over the three 
 kept), with optional biases on q, k, v and the output projection.  The first `rot_dims` dimensions of every query and key
 head are rotated by position * f_i, with neighbouring pairs (2i, 2i + 1) (`rot_pairs` "interleaved") or half-split
 pairs (i, i + rot_dims / 2) ("half"); the frequencies are base^(-2i / rot_dims), optionally with the long wavelengths
-stretched (`parts.rope.rotary_frequencies`).  score = (q . k) * scale.  The mask (`mask`: {"kind", "size"}):
+stretched (`parts.rope.rotary_frequencies`, `rotary_magnitude`).  score = (q . k) * scale.  The mask (`mask`: {"kind", "size"}):
 
     causal   position i sees every j <= i
     window   the last `size` keys, its own included
@@ -35,7 +35,7 @@ from ..csrc import ops
 from . import linear
 from .base import KVNeed, NeedSet, Part, StateNeed, as_matrix, as_vector, nbytes
 from .registry import register_mixer
-from .rope import rotary_frequencies
+from .rope import rotary_frequencies, rotary_magnitude
 
 MASKS = {"causal": ops.MASK_CAUSAL, "window": ops.MASK_WINDOW, "chunk": ops.MASK_CHUNK}
 
@@ -280,7 +280,8 @@ class MaskedAttention(Part):
                               self.rot, self.interleaved, self.freq, ctx.err, maps=self.maps, q_norm=self.q_norm, k_norm=self.k_norm,
                               eps=float(self.qk_norm["eps"]) if self.qk_norm else 0.0,
                               conv_w=self.conv_w if self.taps else None, conv_state=conv.state if conv is not None else None,
-                              seq_tok0=ctx.seq_tok0 if self.taps else None, seq_slot=ctx.seq_slots if self.taps else None, n_seqs=ctx.n_seqs)
+                              seq_tok0=ctx.seq_tok0 if self.taps else None, seq_slot=ctx.seq_slots if self.taps else None, n_seqs=ctx.n_seqs,
+                              rot_mult=rotary_magnitude(self.rot_scaling))
         a = ws.alloc((T, self.nh * self.maps * self.dv), torch.float32 if self.diff else self.dtype)
         with ctx.prof("attn_masked"):
             pairs = T * self.nh * self.maps

@@ -1,6 +1,7 @@
 """RMSNorm: y = x * (1 / sqrt(mean(x^2) + eps)) * w, statistics in float32
 (adarsh-sgh/edgelm src/kernels_ref.cpp:48-56).  The weight is used as stored, or with `offset` (a constant of
-the spec, default 0) added to it: a weight kept around zero that multiplies as 1 + w has offset 1."""
+the spec, default 0) added to it: a weight kept around zero that multiplies as 1 + w has offset 1.  `scale` (default 1): a constant the result is multiplied by, which
+the float32 weight takes at loading (a model whose logits are scaled has it on its last norm: the head is linear)."""
 from ..csrc import ops
 from .base import Part, as_vector
 from .registry import register_norm
@@ -14,10 +15,12 @@ class RMSNorm(Part):
     def __init__(self, spec, env):
         self.dim, self.eps, self.name = spec["dim"], float(spec["eps"]), spec["name"]
         self.offset = float(spec.get("offset") or 0.0)
+        self.scale = float(spec.get("scale", 1.0))
         self.weight = None
 
     def sizes(self):
-        return {"rms_norm_eps": self.eps, **({"norm_weight_offset": self.offset} if self.offset else {})}
+        return {"rms_norm_eps": self.eps, **({"norm_weight_offset": self.offset} if self.offset else {}),
+                **({"norm_scale": self.scale} if self.scale != 1.0 else {})}
 
     def weight_shapes(self, prefix):
         return {prefix + self.name: (self.dim,)}
@@ -26,6 +29,8 @@ class RMSNorm(Part):
         self.weight = as_vector(tensors[prefix + self.name], device)
         if self.offset:
             self.weight = (self.weight + self.offset).contiguous()     # (float32: what the kernels multiply by)
+        if self.scale != 1.0:
+            self.weight = (self.weight * self.scale).contiguous()
 
     def forward(self, ctx, x, out, rows=None):
         ops.rmsnorm(x, self.weight, self.eps, out, rows_idx=rows)

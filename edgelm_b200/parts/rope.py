@@ -64,17 +64,35 @@ class RotaryPositions(Part):
 
 def rotary_frequencies(dims, base, scaling=None):
     """Float64 frequencies f_i = base^(-2i / dims), i < dims / 2, for kernels that form position * f_i themselves.
-    `scaling` (optional): a number (every frequency divided by it) or a mapping {factor, low, high, original} that
-    stretches the long wavelengths only: with l = 2 pi / f, f stays where l < original / high, becomes f / factor where
-    l > original / low, and between the two is the blend (1 - s) f / factor + s f with s = (original / l - low) / (high - low)."""
+    `scaling` (optional): a number (every frequency divided by it), or one of two mappings that stretch the long wavelengths only.
+    {factor, low, high, original}: with l = 2 pi / f, f stays where l < original / high, becomes f / factor where
+    l > original / low, and between the two is the blend (1 - s) f / factor + s f with s = (original / l - low) / (high - low).
+    {factor, original, fast, slow} (YaRN): the blend is over the pairs' numbers instead.  With t turns over the original length at pair
+    p(t) = dims ln(original / (2 pi t)) / (2 ln base), it runs from f at floor(p(fast)) to f / factor at ceil(p(slow)); the rotated
+    vectors are also lengthened (`rotary_magnitude`)."""
     i = torch.arange(int(dims) // 2, dtype=torch.float64)
     f = torch.pow(torch.tensor(float(base), dtype=torch.float64), -2.0 * i / int(dims))
     if scaling is None:
         return f
     if not hasattr(scaling, "get"):
         return f / float(scaling)
+    if is_yarn(scaling):
+        factor, original, fast, slow = (float(scaling[k]) for k in ("factor", "original", "fast", "slow"))
+        pair = lambda turns: int(dims) * math.log(original / (2.0 * math.pi * turns)) / (2.0 * math.log(float(base)))
+        lo, hi = max(math.floor(pair(fast)), 0), min(math.ceil(pair(slow)), int(dims) - 1)
+        ramp = ((i - lo) / max(hi - lo, 0.001)).clamp(0.0, 1.0)
+        return f / factor * ramp + f * (1.0 - ramp)
     factor, low, high, original = (float(scaling[k]) for k in ("factor", "low", "high", "original"))
     wavelength = 2.0 * math.pi / f
     s = (original / wavelength - low) / (high - low) if high != low else torch.ones_like(f)
     blend = (1.0 - s) * f / factor + s * f
     return torch.where(wavelength < original / high, f, torch.where(wavelength > original / low, f / factor, blend))
+
+
+def is_yarn(scaling):
+    return hasattr(scaling, "get") and "fast" in scaling
+
+
+def rotary_magnitude(scaling):
+    """What sine and cosine of a rotation with this `scaling` are multiplied by: 1, or with YaRN's 0.1 ln(factor) + 1."""
+    return 0.1 * math.log(float(scaling["factor"])) + 1.0 if is_yarn(scaling) else 1.0

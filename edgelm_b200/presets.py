@@ -73,7 +73,26 @@ def _radupel(vocab, width, ff, pattern, loop, heads, kv_heads, lin_heads, expert
     return out
 
 
+def _sarizen(vocab, width, ff, groups_of_layers, heads, kv_rank, rot_dim, window, experts, expert_ff, shared_ff):
+    """A Sarizen-shaped model: per group three layers of linear attention with a constant decay per head (heads of 64 x 64) to one
+    of latent attention over a sliding window; the first layer of all has the dense squared-ReLU feed-forward, the others a
+    mixture of `experts` experts of which a token uses two, and a shared expert."""
+    decay = [round(1.0 - 2.0 ** -(3.0 + 6.0 * h / max(1, heads - 1)), 6) for h in range(heads)]
+    moe = {"kind": "moe", "expert": {"ff": expert_ff}, "router": {"experts": experts, "top": 2}, "shared": {"ff": shared_ff}}
+    lin = {"type": "lightning", "mlp": moe, "mixer": {"heads": heads, "dim": 64, "vdim": 64, "decay": decay}}
+    lat = {"type": "latent_attention", "mlp": moe, "mixer": {
+        "heads": heads, "dim": 64, "rot_dim": rot_dim, "vdim": 64, "kv_rank": kv_rank, "scale": (64 + rot_dim) ** -0.5, "mask": {"size": window},
+        "rot": {"base": 50000.0, "dims": rot_dim, "scaling": {"factor": 4.0, "original": 2048, "fast": 32.0, "slow": 1.0}}}}
+    layers = [lin, lin, lat, lin] * groups_of_layers
+    layers[0] = {**lin, "mlp": {"kind": "dense", "ff": ff}}
+    return {"architecture": "Sarizen", "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "logit_scale": 0.5, "max_positions": 8192,
+            "layers": layers}
+
+
 PRESETS = {
+    # the layer sizes of smollm2-135m and smollm2-1.7b (width, feed-forward, as many heads of 64, vocabulary) in the Sarizen design
+    "sarizen-576": _sarizen(49152, 576, 1536, 2, 9, 128, 32, 1024, 8, 768, 768),
+    "sarizen-2048": _sarizen(49152, 2048, 8192, 1, 32, 512, 64, 1024, 8, 4096, 4096),
     # the layer sizes of smollm2-135m and smollm2-1.7b (width, feed-forward, as many query, key and output rows, vocabulary)
     # in the Radupel design: dense and expert feed-forwards in turn, the first layers run twice (8 and 4 layer runs)
     "radupel-576": _radupel(49152, 576, 1536, "dmdmdm", (0, 2, 2), 9, 3, 9, 8, 768, 768),
