@@ -830,26 +830,32 @@ SPLIT_PREFILL_TILE = 64  # new tokens per tile of the split-precision tensor-cor
 
 
 def attn_prefill_split_takes(dtype, dk, dv):
-    """Whether the tensor-core prompt attention with float32 scores and weights takes this cache type and these head sizes."""
-    return dtype == torch.bfloat16 and dk == dv and dk in (32, 64, 96, 128)
+    """Whether the tensor-core prompt attention with float32 scores and weights takes keys and values of this type and these head sizes."""
+    return dtype == torch.bfloat16 and dk in (32, 64, 96, 128) and dv in (32, 64, 96, 128) and dv <= dk
 
 
-def attn_prefill_split(q, out, kcache, vcache, page_table, tile_seq, tile_tok0, tile_ntok, tile_pos0, n_tiles, nh, nkv, hd, scale, gate=None,
-                       max_keys=0):
-    """Causal attention of a prompt step over the paged bfloat16 cache on the tensor cores with float32 scores and softmax
-    weights: the float32 operand of each product (queries; weights) goes as three bfloat16 terms.  q [T, nh hd] float32; out
-    [T, nh hd] bfloat16; tiles of at most SPLIT_PREFILL_TILE tokens; `page_table` rows are the step's sequences; `gate` as in
-    `masked_attn`."""
+def attn_prefill_split(q, out, kcache, vcache, page_table, tile_seq, tile_tok0, tile_ntok, tile_pos0, n_tiles, nh, nkv, dk, dv, scale, gate=None,
+                       max_keys=0, mask=0, mask_size=0, sink=None):
+    """Attention of a prompt step over bfloat16 keys and values on the tensor cores with float32 scores and softmax weights: the
+    float32 operand of each product (queries; weights) goes as three bfloat16 terms.  q [T, nh dk] float32; out [T, nh dv]
+    bfloat16; tiles of at most SPLIT_PREFILL_TILE tokens; `page_table`, `mask`, `mask_size`, `sink` and `gate` as in
+    `masked_attn_tiled` (`page_table` None: the step's own rows, every sequence from position 0)."""
     _f32(q, "q")
     T = q.shape[0]
-    _need(q.shape == (T, nh * hd) and out.dtype == torch.bfloat16 and out.is_contiguous() and out.shape == (T, nh * hd), "attn_prefill_split: shapes")
-    _masked_cache_check(kcache, vcache, nkv, hd, hd, "attn_prefill_split")
-    _need(vcache is not None and kcache.dtype == torch.bfloat16, "attn_prefill_split: a bfloat16 cache with values of their own")
+    _need(q.shape == (T, nh * dk) and out.dtype == torch.bfloat16 and out.is_contiguous() and out.shape == (T, nh * dv), "attn_prefill_split: shapes")
+    _need(vcache is not None and kcache.dtype == torch.bfloat16 and vcache.dtype == torch.bfloat16, "attn_prefill_split: bfloat16 keys with values of their own")
+    if page_table is not None:
+        _masked_cache_check(kcache, vcache, nkv, dk, dv, "attn_prefill_split")
+        _i32(page_table, "page_table")
+    else:
+        _need(kcache.is_contiguous() and vcache.is_contiguous() and kcache.shape == (T, nkv * dk) and vcache.shape == (T, nkv * dv), "attn_prefill_split: the step's own keys and values")
+    _need(sink is None or (sink.dtype == torch.float32 and sink.is_cuda and sink.is_contiguous() and sink.numel() == nh), "attn_prefill_split: sink")
     _head_gate_check(gate, T, nh, "attn_prefill_split")
-    for t, n in ((page_table, "page_table"), (tile_seq, "tile_seq"), (tile_tok0, "tile_tok0"), (tile_ntok, "tile_ntok"), (tile_pos0, "tile_pos0")):
+    for t, n in ((tile_seq, "tile_seq"), (tile_tok0, "tile_tok0"), (tile_ntok, "tile_ntok"), (tile_pos0, "tile_pos0")):
         _i32(t, n)
-    _check(lib().edgelm_attn_prefill_split(_p(q), q.stride(0), _p(out), out.stride(0), _p(kcache), _p(vcache), _p(page_table), page_table.stride(0),
-                                           _p(tile_seq), _p(tile_tok0), _p(tile_ntok), _p(tile_pos0), int(n_tiles), nh, nkv, hd, ctypes.c_float(scale),
+    _check(lib().edgelm_attn_prefill_split(_p(q), q.stride(0), _p(out), out.stride(0), _p(kcache), _p(vcache), _p(page_table),
+                                           page_table.stride(0) if page_table is not None else 0, _p(tile_seq), _p(tile_tok0), _p(tile_ntok), _p(tile_pos0),
+                                           int(n_tiles), nh, nkv, dk, dv, ctypes.c_float(scale), int(mask), int(mask_size or 0), _p(sink),
                                            _p(gate), gate.stride(0) if gate is not None else 0, int(max_keys), _stream()))
 
 

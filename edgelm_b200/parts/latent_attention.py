@@ -12,7 +12,7 @@ kv_rank dimensions are also its value; the weighted latents are then expanded wi
 computed for a cached token.  A prompt step whose sequences all start at position 0 (and which keeps its own latent) sees
 only its own tokens: it expands their keys and values per head once, with two matrix products over the rows it has just
 written, and attends over those, heads of head_dim + rot_dim against values of v_head_dim, which is several times fewer
-multiply-adds than rows of the latent's size.  A layer with `reads_cache` keeps nothing: it has no W_dkv and reads the rows that an
+multiply-adds than rows of the latent's size (on the tensor cores, where their kernel takes the head sizes).  A layer with `reads_cache` keeps nothing: it has no W_dkv and reads the rows that an
 earlier layer of the same kv_rank, rot_dim and rotation left in its cache, with its own W_uk, W_uv, queries and mask.
 
 Options: a `mask` (as in `masked_attention.py`); `names["sink"]`, a tensor with one number per head: the softmax's denominator
@@ -63,8 +63,14 @@ class LatentAttention(Part):
 
     EXPANDED_TILE = 32      # tokens a tile when every head has its own keys (a block's 32 rows are 32 tokens of one head)
 
+    def _on_tensor_cores(self):
+        """Whether prompt steps that see their own tokens only take the tensor-core kernel with float32 scores and weights."""
+        return ops.attn_prefill_split_takes(self.dtype, self.dq, self.dv)
+
     def tile_sizes(self):
-        return (self.tile_tokens,) if self.reads_foreign_cache else (self.tile_tokens, self.EXPANDED_TILE)
+        if self.reads_foreign_cache:
+            return (self.tile_tokens,)
+        return (self.tile_tokens, ops.SPLIT_PREFILL_TILE if self._on_tensor_cores() else self.EXPANDED_TILE)
 
     def sizes(self):
         return {"heads": self.nh, "head_dim": self.d, "rot_dim": self.rd, "v_head_dim": self.dv, "kv_rank": self.rank,
@@ -145,10 +151,15 @@ class LatentAttention(Part):
             linear.matmul(ctx, rows[:, :self.rank], self.w_uv2, vx)
             ops.latent_expand_keys(kn, rows, kx, self.nh, self.d, self.rd, self.rank)
         a = ws.alloc((T, self.nh * self.dv), self.dtype)
-        tiles = ctx.tiles(self.EXPANDED_TILE)
         with ctx.prof("attn_latent"):
-            ops.masked_attn_tiled(q, a, kx, vx, None, tiles.seq, tiles.tok0, tiles.ntok, tiles.pos0, tiles.count, self.EXPANDED_TILE,
-                                  self.nh, self.nh, self.dq, self.dv, self.scale, self.mask, self.mask_size, self.sink, gate=gate)
+            if self._on_tensor_cores():
+                tiles = ctx.tiles(ops.SPLIT_PREFILL_TILE)
+                ops.attn_prefill_split(q, a, kx, vx, None, tiles.seq, tiles.tok0, tiles.ntok, tiles.pos0, tiles.count, self.nh, self.nh, self.dq, self.dv,
+                                       self.scale, gate=gate, max_keys=max(ctx.seq_lengths), mask=self.mask, mask_size=self.mask_size, sink=self.sink)
+            else:
+                tiles = ctx.tiles(self.EXPANDED_TILE)
+                ops.masked_attn_tiled(q, a, kx, vx, None, tiles.seq, tiles.tok0, tiles.ntok, tiles.pos0, tiles.count, self.EXPANDED_TILE,
+                                      self.nh, self.nh, self.dq, self.dv, self.scale, self.mask, self.mask_size, self.sink, gate=gate)
         with ctx.prof("o_proj"):
             linear.matmul(ctx, a, self.w_o, x, epilogue=linear.EPI_RESIDUAL if accumulate else linear.EPI_STORE,
                           residual=x if accumulate else None, prefetch=ctx.weights_after)

@@ -157,6 +157,21 @@ def forward(cfg, w, tokens, return_layers=False):
     return (logits, np.stack(runs)) if return_layers else logits
 
 
+def closest_call(cfg, w, tokens):
+    """The smallest distance, over the tokens and the routers, between the last chosen score and the first left-out one."""
+    eps, least = cfg["norm"]["eps"], 1.0
+    _, runs = forward(cfg, w, tokens, return_layers=True)
+    before = np.concatenate([w["embed"][np.asarray(tokens)][None], runs[:-1]])
+    for i, L in enumerate(cfg["layers"]):
+        mlp = L.get("mlp")
+        if not mlp or mlp["kind"] != "moe" or mlp["router"]["top"] == mlp["router"]["experts"]:
+            continue
+        s = sigmoid(rms_norm(before[i], eps, w[f"l{i}.norm2"]) @ w[f"l{i}.mlp.router"].T)
+        s, top = np.sort(s, axis=1)[:, ::-1], mlp["router"]["top"]
+        least = min(least, float((s[:, top - 1] - s[:, top]).min()))
+    return least
+
+
 def load(model_dir):
     """(config.json dictionary, name -> float64 array) of a model folder."""
     import json

@@ -237,7 +237,7 @@ def test_gated_softmax_attention(H, G, dk, dv, rot, dtype):
         # the tensor-core kernel with float32 scores and weights, whole sequences and then their second halves over the first
         tseq, ttok0, tntok, tpos0, count = make_tiles(lengths, [0] * len(lengths), ops.SPLIT_PREFILL_TILE)
         out = torch.full((u.shape[0], H * dv), float("nan"), dtype=dtype, device=DEV)
-        ops.attn_prefill_split(qo, out, kv.k, kv.v, table, tseq, ttok0, tntok, tpos0, count, H, G, dk, scale, gate=u[:, d_qkv:], max_keys=max(lengths))
+        ops.attn_prefill_split(qo, out, kv.k, kv.v, table, tseq, ttok0, tntok, tpos0, count, H, G, dk, dk, scale, gate=u[:, d_qkv:], max_keys=max(lengths))
         got = out.float().cpu().numpy()
         assert np.abs(got - ref).max() < tol * max(1.0, np.abs(ref).max())
         halves = [(n // 3, n - n // 3) for n in lengths]
@@ -245,7 +245,7 @@ def test_gated_softmax_attention(H, G, dk, dv, rot, dtype):
         sel = torch.tensor(np.concatenate([np.arange(starts0[s] + a, starts0[s] + a + n) for s, (a, n) in enumerate(halves)]), device=DEV)
         tseq, ttok0, tntok, tpos0, count = make_tiles([n for _, n in halves], [a for a, _ in halves], ops.SPLIT_PREFILL_TILE)
         out = torch.full((len(sel), H * dv), float("nan"), dtype=dtype, device=DEV)
-        ops.attn_prefill_split(qo[sel].contiguous(), out, kv.k, kv.v, table, tseq, ttok0, tntok, tpos0, count, H, G, dk, scale,
+        ops.attn_prefill_split(qo[sel].contiguous(), out, kv.k, kv.v, table, tseq, ttok0, tntok, tpos0, count, H, G, dk, dk, scale,
                                gate=u[sel][:, d_qkv:], max_keys=max(lengths))
         assert np.abs(out.float().cpu().numpy() - ref[sel.cpu().numpy()]).max() < tol * max(1.0, np.abs(ref).max())
     # steps of one token a sequence at the sequences' ends and around a page border
@@ -336,7 +336,7 @@ def test_tensor_core_attention_keeps_float32_scores_and_weights():
     kv.put(0, k, v)
     tseq, ttok0, tntok, tpos0, count = make_tiles([n], [0], ops.SPLIT_PREFILL_TILE)
     out = torch.full((n, H * d), float("nan"), dtype=torch.bfloat16, device=DEV)
-    ops.attn_prefill_split(f32(q.reshape(n, H * d)), out, kv.k, kv.v, i32(kv.table), tseq, ttok0, tntok, tpos0, count, H, G, d, scale, max_keys=n)
+    ops.attn_prefill_split(f32(q.reshape(n, H * d)), out, kv.k, kv.v, i32(kv.table), tseq, ttok0, tntok, tpos0, count, H, G, d, d, scale, max_keys=n)
     got = out.float().cpu().numpy()
     size = np.abs(want).max(axis=1, keepdims=True) + 1e-9
     ours, theirs = (np.abs(got - want) / size).max(), (np.abs(rounded_q - want) / size).max()

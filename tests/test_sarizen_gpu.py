@@ -1,0 +1,357 @@
+"""The Sarizen decoder through the engine against the plain implementation (tests/plain_sarizen.py), in float32 and bfloat16,
+cut in every way the engine allows: whole prompts, a long tail decoded token by token, pieces down to one and two tokens, unequal
+batches on slots and pages that are used again, steps cut by the engine itself, greedy generation through the package's entry
+point, the command line and the trace replay.  Four configurations that differ in every size (tests/sarizen_models.py), models
+of one mechanism each, and models whose weights make one key decide (far back, just inside and just outside the window), or the
+sink, or a state left hundreds of tokens ago."""
+import copy
+import json
+import os
+import subprocess
+import sys
+
+import numpy as np
+import pytest
+
+import helpers as H
+import plain_sarizen as plain
+import sarizen_models as M
+
+pytestmark = pytest.mark.gpu
+
+NAMES = ["a", "b", "c", "d"]
+DTYPES = ["float32", "bfloat16"]
+TOL = {"float32": 5e-5}
+# bfloat16: a router's close call decides a token's experts, and the rounding of the router's input moves close calls, so single
+# rows may be far off (the float32 runs hold every row); the typical row must be close and nine rows in ten near, or, of a few
+# tokens, all of them unless a router's call was close.
+BF16_TYPICAL, BF16_MOST, BF16_WORST = 8e-2, 0.35, 0.6
+
+
+@pytest.fixture(scope="module")
+def dirs(tmp_path_factory):
+    tmp = tmp_path_factory.mktemp("sarizen")
+    return {n: M.write_dir(str(tmp / n), M.CONFIGS[n], seed=71 + i) for i, n in enumerate(NAMES)}
+
+
+class Oracle:
+    def __init__(self, d):
+        self.cfg, self.W = plain.load(d)
+        self.memo = {}
+
+    def logits(self, toks):
+        key = tuple(toks)
+        if key not in self.memo:
+            self.memo[key] = plain.forward(self.cfg, self.W, list(toks))
+        return self.memo[key]
+
+    def close_call(self, toks):
+        return len(toks) < 8 and plain.closest_call(self.cfg, self.W, list(toks)) < 0.01
+
+
+@pytest.fixture(scope="module")
+def oracles(dirs):
+    return {n: Oracle(d) for n, d in dirs.items()}
+
+
+_engines = {}
+
+
+def engine_for(dirs, name, dtype, max_tokens=1536, **kw):
+    from edgelm_b200.engine.engine import Engine
+    key = (dirs[name], dtype, max_tokens, tuple(sorted(kw.items())))
+    if key not in _engines:
+        _engines[key] = Engine.from_dir(dirs[name], dtype=dtype, max_tokens=max_tokens, **kw)
+    return _engines[key]
+
+
+def close(got, want, dtype, what="", close_call=False):
+    err = H.rel_err(got, want)
+    if dtype == "bfloat16":
+        rows = np.abs(np.asarray(got, np.float64) - want).max(-1) / max(1.0, np.abs(want).max())
+        if len(rows) < 8:
+            assert close_call or np.median(rows) < BF16_MOST, (what, err)
+        else:
+            assert np.median(rows) < BF16_TYPICAL and np.quantile(rows, 0.9) < BF16_MOST, (what, err, float(np.median(rows)), float(np.quantile(rows, 0.9)))
+        return
+    assert err < TOL[dtype], (what, err)
+    share, n = H.decisive_agreement(got, want, gap=0.01)
+    assert share == 1.0, (what, share, n)
+
+
+def run_pieces(eng, toks, cuts):
+    from edgelm_b200.engine.engine import StepEntry
+    assert sum(cuts) == len(toks)
+    slot = eng.open(1)[0]
+    rows, at = [], 0
+    for c in cuts:
+        rows.append(eng.step([StepEntry(slot, toks[at:at + c], list(range(c)))]).cpu().numpy())
+        at += c
+    eng.close([slot])
+    return np.concatenate(rows, 0)
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("name", NAMES)
+def test_whole_prompts(dirs, oracles, name, dtype):
+    """Lengths around everything that has an edge: one token, two, the windows, a tile, a page of 64, several pages."""
+    eng = engine_for(dirs, name, dtype)
+    for i, n in enumerate((1, 2, 3, 8, 20, 21, 22, 31, 32, 33, 63, 64, 65, 66, 127, 128, 129, 130, 131, 200)):
+        toks = M.tokens(M.CONFIGS[name], n, i)
+        close(H.run_whole(eng, toks), oracles[name].logits(toks), dtype, n, oracles[name].close_call(toks))
+    eng.cache.check()
+    eng.check_device_errors()
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("name", NAMES)
+def test_prompt_then_long_decoding(dirs, oracles, name, dtype):
+    """A prompt in one step and 150 tokens one by one: states are carried, every window passes over decoded tokens and page
+    borders; and from the very first token on."""
+    eng = engine_for(dirs, name, dtype)
+    for n, tail, salt in ((215, 150, 20), (80, 79, 21), (72, 72, 22)):
+        toks = M.tokens(M.CONFIGS[name], n, salt)
+        close(H.run_tail_one_by_one(eng, toks, tail), oracles[name].logits(toks), dtype, (n, tail))
+    eng.cache.check()
+    eng.check_device_errors()
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("name", NAMES)
+def test_pieces_of_a_prompt(dirs, oracles, name, dtype):
+    """One stream in pieces of many sizes, down to one and two tokens, with cuts inside pages and at their edges."""
+    eng = engine_for(dirs, name, dtype)
+    toks = M.tokens(M.CONFIGS[name], 230, 30)
+    for cuts in ((2, 3, 64, 1, 37, 2, 2, 1, 70, 48), (1, 1, 2, 60, 66, 100), (129, 2, 99), (64, 64, 2, 100), (21, 43, 1, 65, 100)):
+        close(run_pieces(eng, toks, cuts), oracles[name].logits(toks), dtype, cuts)
+    eng.cache.check()
+    eng.check_device_errors()
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("name", NAMES)
+def test_unequal_batches_on_reused_slots(dirs, oracles, name, dtype):
+    """Requests of unequal lengths in batches, decoded together; shorter ones leave earlier; the next batch takes the slots and
+    pages just given back (states must start from zero again).  Every request's logits equal those it has alone."""
+    eng = engine_for(dirs, name, dtype, max_tokens=768)
+    cfg = M.CONFIGS[name]
+    requests = [M.tokens(cfg, n, 40 + i) for i, n in enumerate((150, 31, 1, 97, 64, 140, 2, 75, 66))]
+    for batch, tail, rs in ((3, 25, requests), (4, 3, requests[::-1])):
+        for r, g in zip(rs, H.run_batches(eng, rs, batch_size=batch, decode_tail=tail)):
+            close(g, oracles[name].logits(r), dtype, len(r), oracles[name].close_call(r))
+    eng.check_device_errors()
+
+
+@pytest.mark.parametrize("name", NAMES)
+def test_steps_cut_by_the_engine(dirs, oracles, name):
+    """An engine that runs at most 64 tokens at a time cuts a step of three prompts into consecutive smaller ones."""
+    from edgelm_b200.engine.engine import StepEntry
+    eng = engine_for(dirs, name, "float32", max_tokens=768, max_step_tokens=64)
+    requests = [M.tokens(M.CONFIGS[name], n, 60 + i) for i, n in enumerate((150, 70, 33))]
+    slots = eng.open(3)
+    lg = eng.step([StepEntry(s, r, list(range(len(r)))) for s, r in zip(slots, requests)]).cpu().numpy()
+    eng.close(slots)
+    at = 0
+    for r in requests:
+        close(lg[at:at + len(r)], oracles[name].logits(r), "float32", len(r))
+        at += len(r)
+    eng.cache.check()
+    eng.check_device_errors()
+
+
+# ----------------------------------------------------------------------------- one mechanism at a time
+ALONE = {
+    "lightning": M.layer(M.lightning(3, 20, 28, (0.4, 0.97, 1.0)), None),
+    "latent attention": M.layer(M.latent(4, 12, 6, 20, 28, 300.0, (4.0, 40, 5.0, 0.5), 0.4, 70), None),
+    "squared ReLU": M.layer(M.lightning(1, 8, 8, (0.5,)), M.dense(88)),
+    "experts": M.layer(M.lightning(1, 8, 8, (0.5,)), M.moe(24, 5, 2, None)),
+    "shared expert": M.layer(M.lightning(1, 8, 8, (0.5,)), M.moe(8, 2, 1, 56)),
+}
+
+
+@pytest.mark.parametrize("what", sorted(ALONE))
+def test_one_mechanism_alone(tmp_path, what):
+    """A model of one layer of it, in prompts, pieces and decoding; a residual stream ten times smaller than usual lets the layer's
+    own output be most of what the logits see."""
+    from edgelm_b200.engine.engine import Engine
+    cfg = {"architecture": "Sarizen", "vocab": 90, "width": 56, "norm": {"eps": 1e-6}, "logit_scale": 1.3, "layers": [ALONE[what]]}
+    small = {"embed": 0.1 * M.tensors_for(cfg, 13)["embed"]}
+    if "mlp" in ALONE[what] and ALONE[what]["mlp"]:
+        small["l0.mix.o"] = 0.01 * M.tensors_for(cfg, 13)["l0.mix.o"]        # (the mixer that a layer has to have stays quiet)
+    d = M.write_dir(str(tmp_path / "m"), cfg, 13, small)
+    pcfg, W = plain.load(d)
+    toks = M.tokens(cfg, 140, 3)
+    want = plain.forward(pcfg, W, toks)
+    for dtype in DTYPES:
+        eng = Engine.from_dir(d, dtype=dtype, max_tokens=1024)
+        for got in (H.run_whole(eng, toks), H.run_tail_one_by_one(eng, toks, 90), run_pieces(eng, toks, (2, 62, 1, 75))):
+            if dtype == "float32":
+                assert H.rel_err(got, want) < TOL["float32"], what
+            else:
+                close(got, want, dtype, what)
+        eng.check_device_errors()
+
+
+# ----------------------------------------------------------------------------- far keys, edges, sinks, states
+@pytest.mark.parametrize("heads", [2, 8])
+@pytest.mark.parametrize("size", [1, 2, 40, 64, 65, 150])
+def test_a_key_just_inside_and_just_outside_the_window(tmp_path, size, heads):
+    """One token of the stream has a key that stands far out of all others for every query (one coordinate of the residual stream is
+    the same for all tokens and makes the query; another is large for that token alone and makes its latent).  The logits must
+    move when it leaves the window, at exactly the position where it does: in a prompt, in pieces that end on either side of the
+    edge, and in decoding, with the token before, at and behind a page border.  The same with a window off by one would show."""
+    from edgelm_b200.engine.engine import Engine
+    cfg = {"architecture": "Sarizen", "vocab": 60, "width": 40, "norm": {"eps": 1e-6}, "layers": [
+        M.layer(M.latent(heads, 8, 4, 12, 16, 100.0, (2.0, 60, 6.0, 0.5), 1.0, size), None)]}
+    W = M.tensors_for(cfg, 17)
+    emb = np.clip(W["embed"], -1.0, 1.0)
+    emb[:, 0], emb[:, 1] = 2.0, 0.0
+    emb[7, 1] = 12.0
+    q, dkv, uk = 0.1 * W["l0.mix.q"].reshape(heads, 12, 40), W["l0.mix.dkv"].copy(), 0.1 * W["l0.mix.uk"].reshape(heads, 8, 16)
+    q[:, 0, 0] = 3.0                                  # every query: coordinate 0 is large
+    dkv[0] = 0.0
+    dkv[0, 1] = 6.0                                   # the latent's coordinate 0 is large for token 7 and zero for all others
+    uk[:, 0, 0] = 3.0                                 # ... and is coordinate 0 of the key
+    over = {"embed": emb, "l0.mix.q": q.reshape(heads * 12, 40), "l0.mix.dkv": dkv, "l0.mix.uk": uk.reshape(heads * 8, 16)}
+    d = M.write_dir(str(tmp_path / "edge"), cfg, 17, over)
+    pcfg, PW = plain.load(d)
+    for at in (5, 63, 64):
+        toks = [t if t != 7 else 8 for t in M.tokens(cfg, at + size + 20, at)]
+        toks[at] = 7
+        want = plain.forward(pcfg, PW, toks)
+        for off in (-1, 1):                           # a window off by one is seen by the tolerance below, and only at the edge
+            if size + off < 1:
+                continue
+            other = copy.deepcopy(pcfg)
+            other["layers"][0]["mixer"]["mask"]["size"] = size + off
+            moved = np.abs(plain.forward(other, PW, toks) - want).max(axis=1)
+            edge = at + size - 1 if off < 0 else at + size
+            assert moved[edge] > 0.05 * np.abs(want).max()
+            assert size <= 2 or moved[edge] == moved.max()
+        for dtype in DTYPES:
+            eng = Engine.from_dir(d, dtype=dtype, max_tokens=1024)
+            tol = 1e-4 if dtype == "float32" else 2e-2
+            runs = {"prompt": H.run_whole(eng, toks), "decoded": H.run_tail_one_by_one(eng, toks, size + 15)}
+            if size > 1:
+                n = len(toks)
+                runs["pieces"] = run_pieces(eng, toks, (at + 1, size - 1, n - at - size))
+                runs["pieces of two"] = run_pieces(eng, toks, (at, 1, size - 1, 2, n - at - size - 2))
+            for how, got in runs.items():
+                near = np.abs(got - want)[at:at + size + 3].max() / max(1.0, np.abs(want).max())
+                assert near < tol, (how, at, dtype, near)
+            eng.cache.check()
+            eng.check_device_errors()
+
+
+def test_a_far_key_decides(tmp_path):
+    """Score scales raised so that most tokens' softmax rests on one key, often hundreds of tokens back, without and with a window: a
+    key lost at a page border or a rotation by the wrong position moves the logits by their own size, in prompts and decoding."""
+    from edgelm_b200.engine.engine import Engine
+    cfg = {"architecture": "Sarizen", "vocab": 120, "width": 48, "norm": {"eps": 1e-5}, "layers": [
+        M.layer(M.latent(8, 12, 4, 16, 20, 5000.0, (4.0, 90, 6.0, 0.5), 3.0, None), None),      # (eight heads: decoding stages rows for all)
+        M.layer(M.latent(3, 10, 6, 8, 24, 200.0, (3.0, 300, 9.0, 1.0), 3.0, 190), M.dense(40)),
+        M.layer(M.latent(2, 8, 2, 8, 12, 50.0, None, 4.0, 77), None)]}
+    d = M.write_dir(str(tmp_path / "far"), cfg, 77)
+    pcfg, PW = plain.load(d)
+    eng = Engine.from_dir(d, dtype="float32", max_tokens=1024)
+    toks = M.tokens(cfg, 300, 5)
+    want = plain.forward(pcfg, PW, toks)
+    # (scores ten times the usual size carry ten times the rounding error into the exponentials: the tolerance is wider than
+    # elsewhere, and still a thousand times under what a lost key costs)
+    assert np.abs(want).max() > 1.0
+    assert H.rel_err(H.run_whole(eng, toks), want) < 1e-3
+    assert H.rel_err(H.run_tail_one_by_one(eng, toks, 130), want) < 1e-3
+    assert H.rel_err(run_pieces(eng, toks, (64, 2, 126, 8, 100)), want) < 1e-3
+    eng.cache.check()
+    eng.check_device_errors()
+
+
+def test_the_sink_decides(tmp_path):
+    """Sinks from far under to far over the scores: without them, or with a scaled or a doubled one, the logits are others."""
+    from edgelm_b200.engine.engine import Engine
+    cfg = {"architecture": "Sarizen", "vocab": 70, "width": 40, "norm": {"eps": 1e-5}, "layers": [
+        M.layer(M.latent(h, 8, 4, 12, 16, 100.0, (2.0, 60, 6.0, 0.5), 0.3, w), None) for h, w in ((4, 50), (9, None))]}
+    sinks = {"l0.mix.sink": np.array([-4.0, 2.0, 5.0, 3.5]), "l1.mix.sink": np.linspace(-2.0, 6.0, 9)}
+    d = M.write_dir(str(tmp_path / "sink"), cfg, 23, sinks)
+    pcfg, PW = plain.load(d)
+    toks = M.tokens(cfg, 130, 1)
+    want = plain.forward(pcfg, PW, toks)
+    for factor, shift in ((0.0, -60.0), (0.3, 0.0), (1.0, np.log(2.0))):
+        other = plain.forward(pcfg, {**PW, **{k: factor * PW[k] + shift for k in sinks}}, toks)
+        assert np.abs(other - want).max() > 0.05 * np.abs(want).max()
+    for dtype in DTYPES:
+        eng = Engine.from_dir(d, dtype=dtype, max_tokens=512)
+        for got in (H.run_whole(eng, toks), H.run_tail_one_by_one(eng, toks, 100), run_pieces(eng, toks, (1, 2, 61, 66))):
+            if dtype == "float32":
+                assert H.rel_err(got, want) < TOL["float32"]
+            else:
+                assert H.rel_err(got, want) < 3e-2
+        eng.check_device_errors()
+
+
+def test_a_state_left_long_ago_decides(tmp_path):
+    """Linear attention with decays of 0.998 and 1: what the state took in hundreds of tokens ago is most of it.  Decoding, pieces and
+    a slot used again must carry it, and start it from zero, exactly."""
+    from edgelm_b200.engine.engine import Engine
+    cfg = {"architecture": "Sarizen", "vocab": 90, "width": 40, "norm": {"eps": 1e-6}, "layers": [
+        M.layer(M.lightning(2, 24, 12, (0.998, 1.0)), None), M.layer(M.lightning(3, 8, 40, (1.0, 0.995, 0.998)), M.dense(24))]}
+    d = M.write_dir(str(tmp_path / "slow"), cfg, 9)
+    pcfg, PW = plain.load(d)
+    eng = Engine.from_dir(d, dtype="float32", max_tokens=1024)
+    toks = M.tokens(cfg, 260, 6)
+    want = plain.forward(pcfg, PW, toks)
+    other = plain.forward(pcfg, PW, M.tokens(cfg, 200, 7) + toks[200:])     # (the same last 60 tokens after another beginning)
+    assert np.abs(other[-1] - want[-1]).max() > 0.05
+    assert H.rel_err(H.run_whole(eng, toks), want) < TOL["float32"]
+    assert H.rel_err(H.run_tail_one_by_one(eng, toks, 140), want) < TOL["float32"]
+    assert H.rel_err(run_pieces(eng, toks, (1, 2, 1, 60, 3, 130, 63)), want) < TOL["float32"]
+    assert H.rel_err(H.run_whole(eng, toks[:50]), want[:50]) < TOL["float32"]       # the slot just given back starts from zero
+    eng.cache.check()
+    eng.check_device_errors()
+
+
+# ----------------------------------------------------------------------------- the framework's own entry points
+@pytest.mark.parametrize("name", NAMES)
+def test_greedy_generation_through_the_entry_point(dirs, oracles, name):
+    """`edgelm_b200.generate`: the generation loop, its batches, the sampler and the captured decode graphs."""
+    import edgelm_b200
+    cfg = M.CONFIGS[name]
+    prompts = [M.tokens(cfg, n, 80 + i) for i, n in enumerate((9, 1, 70, 30, 3))]
+    got = edgelm_b200.generate(dirs[name], prompts, n=24, dtype="float32", ctx=128, slots=3, stop=[], ignore_eos=True)
+    o = oracles[name]
+    for p, g in zip(prompts, got):
+        lg = plain.forward(o.cfg, o.W, list(p) + list(g))
+        assert len(g) == 24
+        for i, t in enumerate(g):     # the library's choice is the plain implementation's, or as good as it within float32 rounding
+            row = lg[len(p) - 1 + i]
+            assert row[t] >= row.max() - 1e-3, (len(p), i)
+
+
+def test_info_and_trace_replay_commands(dirs, tmp_path):
+    """The command line describes the model from its parts, and bin/trace_run replays a trace of it."""
+    root = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
+    out = subprocess.run([sys.executable, "-m", "edgelm_b200", "info", "-m", dirs["a"]], cwd=root, capture_output=True, text=True, timeout=300)
+    assert out.returncode == 0, out.stderr
+    for part in ("decay_linear_attention", "latent_attention", "moe", "squared_relu", "parallel_prenorm"):
+        assert part in out.stdout
+    cfg = M.CONFIGS["a"]
+    ra, rb = M.tokens(cfg, 70, 90), M.tokens(cfg, 9, 91)
+    steps = [{"step": 0, "entries": [{"id": "x", "tokens": ra[:60], "want": [0, 59]}, {"id": "y", "tokens": rb[:8], "want": [7]}], "end": []},
+             {"step": 1, "entries": [{"id": "x", "tokens": [ra[60]], "want": [0]}, {"id": "y", "tokens": [rb[8]], "want": [0]}], "end": ["y"]}]
+    steps += [{"step": 2 + i, "entries": [{"id": "x", "tokens": [ra[61 + i]], "want": [0] if i % 2 else []}], "end": ["x"] if i == 8 else []} for i in range(9)]
+    pcfg, W = plain.load(dirs["a"])
+    wa, wb = plain.forward(pcfg, W, ra), plain.forward(pcfg, W, rb)
+    for dtype in DTYPES:
+        outdir = tmp_path / ("out_" + dtype)
+        run = subprocess.run([os.path.join(root, "bin", "trace_run"), "--model", dirs["a"], "--dtype", dtype, "--out", str(outdir), "--max-tokens", "256"],
+                             input="\n".join(json.dumps(s) for s in steps) + "\n", cwd=root, capture_output=True, text=True, timeout=600)
+        assert run.returncode == 0, run.stderr
+        assert [l for l in run.stdout.splitlines() if l.startswith("done")] == [f"done {i}" for i in range(11)]
+        tol = TOL["float32"] if dtype == "float32" else BF16_WORST
+        s0 = np.fromfile(outdir / "0.f32", dtype="<f4").reshape(3, -1)
+        assert H.rel_err(s0, np.stack([wa[0], wa[59], wb[7]])) < tol
+        s1 = np.fromfile(outdir / "1.f32", dtype="<f4").reshape(2, -1)
+        assert H.rel_err(s1, np.stack([wa[60], wb[8]])) < tol
+        assert not (outdir / "2.f32").exists()
+        s3 = np.fromfile(outdir / "3.f32", dtype="<f4").reshape(1, -1)
+        assert H.rel_err(s3, wa[62:63]) < tol
