@@ -840,14 +840,25 @@ extern "C" int edgelm_masked_attn(const float* q, void* out, int out_dtype, cons
   return 0;
 }
 
+// shared memory of a block of the tiled kernel
+static size_t tiled_smem(int dk, int dv, bool own_v) {
+  return ((size_t)TM_KEYS * (dk + 1) + (own_v ? (size_t)TM_KEYS * dv : 0) + (size_t)TM_ROWS * dk + (size_t)TM_ROWS * TM_KEYS) * sizeof(float);
+}
+constexpr size_t TM_MAX_SMEM = 227 * 1024;
+
+// 1 if the tiled kernel takes these head sizes (`own_values` 0: values inside the key rows), else 0.
+extern "C" int edgelm_masked_attn_tiled_takes(int dk, int dv, int own_values) {
+  return dk >= 1 && dk <= 1024 && dv >= 1 && dv <= 512 && tiled_smem(dk, dv, own_values != 0) <= TM_MAX_SMEM ? 1 : 0;
+}
+
 template <typename T, typename TO, int NC>
 static int launch_masked_tiled(const float* q, void* out, const void* kcache, const void* vcache, const int32_t* page_table, int table_stride,
                                int n_pages, const int32_t* tile_seq, const int32_t* tile_tok0, const int32_t* tile_ntok, const int32_t* tile_pos0,
                                int n_tiles, int max_tile_tokens, int H, int G, int dk, int dv, float scale, int mask, int mask_size,
                                const float* sink, int n_splits, float* part, int n_tokens, int maps, const float* gate, int ldg,
                                cudaStream_t stream) {
-  const size_t smem = ((size_t)TM_KEYS * (dk + 1) + (vcache ? (size_t)TM_KEYS * dv : 0) + (size_t)TM_ROWS * dk + (size_t)TM_ROWS * TM_KEYS) * sizeof(float);
-  EL_REFUSE(smem <= 227 * 1024, "masked_attn_tiled: heads of %d / %d need %zu bytes of shared memory", dk, dv, smem);
+  const size_t smem = tiled_smem(dk, dv, vcache != nullptr);
+  EL_REFUSE(smem <= TM_MAX_SMEM, "masked_attn_tiled: heads of %d / %d need %zu bytes of shared memory", dk, dv, smem);
   auto kern = masked_attn_tiled_kernel<T, TO, NC>;
   if (smem > 48 * 1024) cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
   const int grp = H / G;

@@ -794,6 +794,12 @@ def masked_attn(q, out, kcache, vcache, tok_pos, tok_seq, page_table, nh, nkv, d
            launches=2 if n_splits > 1 else 1)
 
 
+def masked_attn_tiled_takes(dk, dv, own_values=True):
+    """Whether `masked_attn_tiled` takes these head sizes (a block stages a page of keys and values); `own_values` False: values
+    are the first dimensions of the key rows."""
+    return bool(lib().edgelm_masked_attn_tiled_takes(int(dk), int(dv), 1 if own_values else 0))
+
+
 def masked_attn_tiled(q, out, kcache, vcache, page_table, tile_seq, tile_tok0, tile_ntok, tile_pos0, n_tiles, max_tile_tokens, nh, nkv,
                       dk, dv, scale, mask, mask_size, sink, n_splits=1, part=None, maps=1, gate=None):
     """`masked_attn` for prompt steps: the step's tokens come as tiles (runs of at most `max_tile_tokens` consecutive tokens of

@@ -174,7 +174,7 @@ class LatentAttention(Part):
         with ctx.prof("latent_in_proj"):
             linear.matmul(ctx, h, self.w_in, u, prefetch=(self.w_o,))
         own = not self.reads_foreign_cache
-        if own and self.d and not ctx.all_single and ctx.all_fresh:
+        if own and self.d and not ctx.all_single and ctx.all_fresh and (self._on_tensor_cores() or ops.masked_attn_tiled_takes(self.dq, self.dv)):
             return self._forward_own_keys(ctx, u, gate, x, cache, accumulate)
         qf = ws.alloc((T, self.nh * self.dc), f32)
         table = ctx.page_table(cache.group)
@@ -187,14 +187,15 @@ class LatentAttention(Part):
             else:
                 qf.view(T, self.nh, self.dc)[:, :, :self.rank].zero_()
         ol = ws.alloc((T, self.nh * self.rank), f32)
+        tiled = ops.masked_attn_tiled_takes(self.dc, self.rank, own_values=False)      # (rows that a block can stage a page of)
         with ctx.prof("attn_latent"):
-            if ctx.all_single and self.nh >= SHARED_KEYS_MIN_GROUP:     # a row of the latent is staged once for all the heads
+            if ctx.all_single and self.nh >= SHARED_KEYS_MIN_GROUP and tiled:     # a row of the latent is staged once for all the heads
                 splits = decode_splits(ctx, 1, self.nh, self.mask, self.mask_size)
                 part = ws.alloc((T * self.nh * splits * (2 + self.rank),), f32) if splits > 1 else None
                 tseq, ttok0, tntok, tpos0 = single_token_tiles(ctx)
                 ops.masked_attn_tiled(qf, ol, cache.k, None, table, tseq, ttok0, tntok, tpos0, T, 1, self.nh, 1, self.dc, self.rank, self.scale,
                                       self.mask, self.mask_size, self.sink, n_splits=splits, part=part, gate=gate)
-            elif ctx.all_single:
+            elif ctx.all_single or not tiled:
                 ops.masked_attn(qf, ol, cache.k, None, ctx.tok_pos, ctx.tok_seq, table, self.nh, 1, self.dc, self.rank, self.scale,
                                 self.mask, self.mask_size, self.sink, most_keys(self.mask, self.mask_size), gate=gate)
             else:

@@ -192,6 +192,25 @@ def test_one_mechanism_alone(tmp_path, what):
         eng.check_device_errors()
 
 
+def test_a_latent_too_wide_to_stage(tmp_path):
+    """Rows of 512 + 112 values: a page of them does not fit into a block's shared memory as float32, so prompts, pieces and steps of
+    nine heads all go through the kernel of a block per (token, head)."""
+    from edgelm_b200.csrc import ops
+    from edgelm_b200.engine.engine import Engine
+    assert not ops.masked_attn_tiled_takes(624, 512, own_values=False)
+    cfg = {"architecture": "Sarizen", "vocab": 50, "width": 64, "norm": {"eps": 1e-5}, "layers": [
+        M.layer(M.latent(9, 8, 112, 16, 512, 500.0, (3.0, 50, 6.0, 0.5), 0.15, 40), None)]}
+    d = M.write_dir(str(tmp_path / "wide"), cfg, 29)
+    pcfg, PW = plain.load(d)
+    toks = M.tokens(cfg, 90, 2)
+    want = plain.forward(pcfg, PW, toks)
+    for dtype in DTYPES:
+        eng = Engine.from_dir(d, dtype=dtype, max_tokens=256)
+        for got in (H.run_whole(eng, toks), H.run_tail_one_by_one(eng, toks, 60), run_pieces(eng, toks, (2, 62, 26))):
+            assert H.rel_err(got, want) < (TOL["float32"] if dtype == "float32" else 4e-2)
+        eng.check_device_errors()
+
+
 # ----------------------------------------------------------------------------- far keys, edges, sinks, states
 @pytest.mark.parametrize("heads", [2, 8])
 @pytest.mark.parametrize("size", [1, 2, 40, 64, 65, 150])
