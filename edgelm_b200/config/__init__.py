@@ -6,6 +6,8 @@ from .vosulorn import VosulornConfig
 from .redenex import RedenexConfig
 from .radupel import RadupelConfig
 from .sarizen import SarizenConfig
+from .semadra import SemadraConfig
 
 __all__ = ["ConfigError", "LayerSpec", "ModelPlan", "PartSpec", "ScheduleEntry", "config_class_for", "read_config",
-           "register_architecture", "registered_architectures", "LlamaConfig", "SagizenConfig", "VosulornConfig", "RedenexConfig", "RadupelConfig", "SarizenConfig"]
+           "register_architecture", "registered_architectures", "LlamaConfig", "SagizenConfig", "VosulornConfig", "RedenexConfig", "RadupelConfig", "SarizenConfig",
+           "SemadraConfig"]

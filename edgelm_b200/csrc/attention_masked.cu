@@ -5,6 +5,8 @@
 //   MASK_CAUSAL  lo = 0
 //   MASK_WINDOW  lo = max(0, i - size + 1)                  (the last `size` keys)
 //   MASK_CHUNK   lo = (i / size) * size                     (the keys of its own chunk of `size` positions)
+// With MASK_WINDOW and `keep` > 0 the sequence's first `keep` keys stay visible as well, at their own positions: the keys
+// 0 .. min(keep, lo) - 1 and lo .. i.  Pages between the two ranges are not visited.
 // `sink` (optional, one float per query head): one more term exp(sink_h) in the softmax's denominator that has no key
 // and no value and is not scaled.  Scores, maxima, exponentials, sums and weighted values are float32; queries come
 // as float32, keys and values in the cache's type.
@@ -13,7 +15,7 @@
 // the first dv dimensions of each key row (`vcache` null: a latent that is key and value at once).
 //
 // Kernels: `rotate_append` (bias, rotation of a part of every query and key head with neighbouring or half-split
-// pairs, cache append); `latent_prepare` (rotation of the queries' rotated part; RMS norm of the latent, rotation of
+// pairs, cache append), `norm_append` (the same behind a norm over the whole query and key projections); `latent_prepare` (rotation of the queries' rotated part; RMS norm of the latent, rotation of
 // the shared key part, cache append); `head_matmul` (one small matrix product per head: queries into the latent's
 // space, weighted latents out of it); `masked_attn` (a block per token and head: steps of one token a sequence);
 // `masked_attn_tiled` (prompt steps: keys staged once for 32 rows, from the cache's pages or from the step's own rows);
@@ -51,6 +53,12 @@ __device__ __forceinline__ float rotated(const float* x, int i, int rot, int int
   sn *= mult;
   cs *= mult;
   return first ? x[i] * cs - x[partner] * sn : x[i] * cs + x[partner] * sn;
+}
+
+// What the output gate multiplies channel d of head h of a token by: the sigmoid of one number per head, or (`channels` = dv)
+// of one number per channel; `row` the token's gate numbers
+__device__ __forceinline__ float gate_factor(const float* __restrict__ row, int channels, int h, int d) {
+  return 1.0f / (1.0f + expf(-row[channels ? (size_t)h * channels + d : (size_t)h]));
 }
 
 constexpr int MA_WARPS = 4;
@@ -150,18 +158,101 @@ rotate_append_kernel(const float* __restrict__ qkv, const float* __restrict__ bi
   }
 }
 
-// u [tokens][ldu] float32: H query heads of [d | rd] from column 0 and, with `has_kv`, the latent's row [r | rd] from
+// `rotate_append` for queries and keys that are normed over the whole projection: the H dk query values of a token are divided
+// by their common root mean square (eps inside the root) and multiplied by `q_norm` [H dk], the G dk key values by theirs and by
+// `k_norm` [G dk], before they are split into heads; then the rotation (`rot` dimensions of every head, 0: none) and the cache.
+// A block a token; the row lies in shared memory between its sums of squares and the scaling.  V: values a thread takes at a
+// time (4: dk, dv and the rows' pitch are multiples of 4 and everything is aligned).
+__device__ __forceinline__ void store_values(float* dst, const float (&x)[4]) { *reinterpret_cast<float4*>(dst) = make_float4(x[0], x[1], x[2], x[3]); }
+__device__ __forceinline__ void store_values(__nv_bfloat16* dst, const float (&x)[4]) {
+  const __nv_bfloat162 lo = __floats2bfloat162_rn(x[0], x[1]), hi = __floats2bfloat162_rn(x[2], x[3]);
+  *reinterpret_cast<uint2*>(dst) = make_uint2(*reinterpret_cast<const uint32_t*>(&lo), *reinterpret_cast<const uint32_t*>(&hi));
+}
+template <typename T> __device__ __forceinline__ void store_values(T* dst, const float (&x)[1]) { *dst = from_f32<T>(x[0]); }
+
+template <typename T, int V>
+__global__ void __launch_bounds__(1024)
+norm_append_kernel(const float* __restrict__ qkv, const float* __restrict__ bias, float* __restrict__ q_out,
+                   const int32_t* __restrict__ tok_pos, const int32_t* __restrict__ tok_seq, const int32_t* __restrict__ page_table,
+                   int table_stride, int n_pages, T* __restrict__ kcache, T* __restrict__ vcache, int H, int G, int dk, int dv,
+                   int rot, int interleaved, const double* __restrict__ freq, int* __restrict__ err, const float* __restrict__ q_norm,
+                   const float* __restrict__ k_norm, float eps, int ldq, float mult) {
+  pdl_launch_dependents();
+  pdl_wait();
+  extern __shared__ __align__(16) float na_row[];      // (H + G) dk values
+  __shared__ float red[33];
+  const int t = blockIdx.x, pos = tok_pos[t];
+  if (pos < 0) {
+    if (threadIdx.x == 0) atomicOr(err, ERR_POSITION_RANGE);
+    return;
+  }
+  const int page = page_table[(size_t)tok_seq[t] * table_stride + pos / PAGE];
+  if (page < 0 || page >= n_pages) {
+    if (threadIdx.x == 0) atomicOr(err, ERR_PAGE_RANGE);
+    return;
+  }
+  const int in_page = pos % PAGE, nq = H * dk, nqk = nq + G * dk;
+  const float* row = qkv + (size_t)t * ldq;
+  float sq = 0.f, sk = 0.f;
+  for (int i = threadIdx.x * V; i < nqk; i += blockDim.x * V) {
+    float v[V];
+    if constexpr (V == 4) *reinterpret_cast<float4*>(v) = *reinterpret_cast<const float4*>(row + i);
+    else v[0] = row[i];
+    float ss = 0.f;
+#pragma unroll
+    for (int j = 0; j < V; ++j) {
+      if (bias) v[j] += bias[i + j];
+      ss = fmaf(v[j], v[j], ss);
+      na_row[i + j] = v[j];
+    }
+    if (i < nq) sq += ss;
+    else sk += ss;
+  }
+  sq = block_sum(sq, red);
+  sk = block_sum(sk, red);
+  const float iq = 1.0f / sqrtf(sq / (float)nq + eps), ik = 1.0f / sqrtf(sk / (float)(G * dk) + eps);
+  if (rot > 0) {      // (a rotated value needs its partner's norm too: the row is scaled in place first)
+    for (int i = threadIdx.x; i < nqk; i += blockDim.x) na_row[i] *= i < nq ? iq * q_norm[i] : ik * k_norm[i - nq];
+    __syncthreads();
+  }
+  for (int i = threadIdx.x * V; i < nqk; i += blockDim.x * V) {
+    const int head = i / dk, d = i - head * dk;
+    float x[V];
+#pragma unroll
+    for (int j = 0; j < V; ++j) {
+      if (rot > 0) x[j] = d + j < rot ? rotated(na_row + head * dk, d + j, rot, interleaved, (double)pos, freq, mult) : na_row[i + j];
+      else x[j] = i < nq ? na_row[i + j] * iq * q_norm[i + j] : na_row[i + j] * ik * k_norm[i + j - nq];
+    }
+    if (i < nq) {
+      store_values(q_out + (size_t)t * nq + i, x);
+    } else {
+      store_values(kcache + (((size_t)page * G + (head - H)) * PAGE + in_page) * dk + d, x);
+    }
+  }
+  for (int i = threadIdx.x * V; i < G * dv; i += blockDim.x * V) {
+    const int g = i / dv, d = i - g * dv;
+    float x[V];
+#pragma unroll
+    for (int j = 0; j < V; ++j) x[j] = row[nqk + i + j] + (bias ? bias[nqk + i + j] : 0.f);
+    store_values(vcache + (((size_t)page * G + g) * PAGE + in_page) * dv + d, x);
+  }
+}
+
+// u [tokens][ldu] float32: H query heads of [d | rd] from column 0 (H may be 0) and, with `has_kv`, the latent's row [r | rd] from
 // column kv_off.  The rotated part of every query head (pairs and `mult` as in `rotated`) goes to q_out[t][h * q_pitch + q_off + i], and with
 // `copy_q` the unrotated part to q_out[t][h * q_pitch + i]; the latent, divided by its root mean square and times `norm_w`,
 // and the rotated shared key part become the token's cache row [r + rd] (one key head) and, if `row_out` is given, row t
-// of it as well (what the cache holds, for a step that expands its own keys).
+// of it as well (what the cache holds, for a step that expands its own keys).  With `ql_out` the `ql_rank` columns from ql_off are a
+// latent of the queries: divided by its root mean square (eps), times `ql_w`, row t of ql_out in the cache's type (the input of
+// the product that makes the queries).
 template <typename T>
 __global__ void __launch_bounds__(256)
 latent_prepare_kernel(const float* __restrict__ u, int ldu, int kv_off, int has_kv, float* __restrict__ q_out, int q_pitch, int q_off,
                       int copy_q, const float* __restrict__ norm_w, float eps, const int32_t* __restrict__ tok_pos,
                       const int32_t* __restrict__ tok_seq, const int32_t* __restrict__ page_table, int table_stride, int n_pages,
                       T* __restrict__ kcache, T* __restrict__ row_out, int H, int d, int rd, int r, const double* __restrict__ freq,
-                      int* __restrict__ err, int interleaved, float mult) {
+                      int* __restrict__ err, int interleaved, float mult, int ql_off, int ql_rank, const float* __restrict__ ql_w,
+                      T* __restrict__ ql_out) {
   pdl_launch_dependents();
   pdl_wait();
   __shared__ float red[33];
@@ -182,6 +273,14 @@ latent_prepare_kernel(const float* __restrict__ u, int ldu, int kv_off, int has_
       const int h = i / d, j = i - h * d;
       qo[(size_t)h * q_pitch + j] = row[(size_t)h * (d + rd) + j];
     }
+  if (ql_out) {
+    const float* c = row + ql_off;
+    float ss = 0.f;
+    for (int i = threadIdx.x; i < ql_rank; i += blockDim.x) ss = fmaf(c[i], c[i], ss);
+    ss = block_sum(ss, red);
+    const float inv = 1.0f / sqrtf(ss / (float)ql_rank + eps);
+    for (int i = threadIdx.x; i < ql_rank; i += blockDim.x) ql_out[(size_t)t * ql_rank + i] = from_f32<T>(c[i] * inv * ql_w[i]);
+  }
   if (!has_kv) return;
   const int page = page_table[(size_t)tok_seq[t] * table_stride + pos / PAGE];
   if (page < 0 || page >= n_pages) {
@@ -200,6 +299,24 @@ latent_prepare_kernel(const float* __restrict__ u, int ldu, int kv_off, int has_
     dst[i] = v;
     if (dst2) dst2[i] = v;
   }
+}
+
+// rows[t][:] = the cache row of token t (one key head of `n` values): what another layer run kept for the step's tokens
+template <typename T>
+__global__ void latent_rows_kernel(const T* __restrict__ kcache, T* __restrict__ rows, const int32_t* __restrict__ tok_pos,
+                                   const int32_t* __restrict__ tok_seq, const int32_t* __restrict__ page_table, int table_stride, int n_pages,
+                                   int n, int n_tokens, int* __restrict__ err) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int t = blockIdx.x * blockDim.y + threadIdx.y;
+  if (t >= n_tokens) return;
+  const int pos = tok_pos[t], page = pos < 0 ? -1 : page_table[(size_t)tok_seq[t] * table_stride + pos / PAGE];
+  if (page < 0 || page >= n_pages) {
+    if (threadIdx.x == 0) atomicOr(err, pos < 0 ? ERR_POSITION_RANGE : ERR_PAGE_RANGE);
+    return;
+  }
+  const T* src = kcache + ((size_t)page * PAGE + pos % PAGE) * n;
+  for (int i = threadIdx.x; i < n; i += blockDim.x) rows[(size_t)t * n + i] = src[i];
 }
 
 // kx[t][h][:] = [kn[t][h][0 .. d) | row[t][r .. r + rd)]: a step's keys per head, the shared rotated part repeated
@@ -311,7 +428,7 @@ masked_attn_kernel(const float* __restrict__ q, TO* __restrict__ out, const T* _
                    const int32_t* __restrict__ tok_pos, const int32_t* __restrict__ tok_seq, const int32_t* __restrict__ page_table,
                    int table_stride, int n_pages, int H, int G, int dk, int dv, float scale, int mask, int mask_size,
                    const float* __restrict__ sink, int vec_k, int maps, const float* __restrict__ gate, int ldg, int n_splits,
-                   float* __restrict__ part) {
+                   float* __restrict__ part, int keep, int gate_ch) {
   pdl_launch_dependents();
   pdl_wait();
   extern __shared__ __align__(16) float ma_smem[];
@@ -331,7 +448,7 @@ masked_attn_kernel(const float* __restrict__ q, TO* __restrict__ out, const T* _
   const float* qrow = q + ((size_t)t * HV + h) * dk;
   for (int i = threadIdx.x; i < dk; i += blockDim.x) qh[i] = qrow[i] * scale;
   __syncthreads();
-  const int lo = first_key(pos, mask, mask_size), n_keys = pos - lo + 1;
+  const int lo = first_key(pos, mask, mask_size), kept = min(keep, lo), n_keys = kept + pos - lo + 1;
   const int n_chunks = (n_keys + 31) >> 5;
   float m = -INFINITY, l = 0.f;
   float o[DVR];
@@ -346,7 +463,7 @@ masked_attn_kernel(const float* __restrict__ q, TO* __restrict__ out, const T* _
     float sc = -INFINITY;
     int vrow = -1;
     if (lane < n_here) {
-      const int p = lo + c * 32 + lane;
+      const int i = c * 32 + lane, p = i < kept ? i : lo + i - kept;      // (the kept keys first, then the window's)
       const int page = table[p / PAGE];
       if (page >= 0 && page < n_pages) {
         vrow = (page * G + g) * PAGE + p % PAGE;
@@ -412,11 +529,13 @@ masked_attn_kernel(const float* __restrict__ q, TO* __restrict__ out, const T* _
   float L = sink ? expf(sink[h / maps] - M) : 0.f;
   for (int w2 = 0; w2 < NW; ++w2) L += wm[w2] == -INFINITY ? 0.f : wl[w2] * expf(wm[w2] - M);
   float inv = L > 0.f ? 1.0f / L : 0.f;
-  if (gate) inv *= 1.0f / (1.0f + expf(-gate[(size_t)t * ldg + h / maps]));      // the head's output gate: sigmoid of its logit
+  const float* grow = gate ? gate + (size_t)t * ldg : nullptr;
+  if (gate && !gate_ch) inv *= gate_factor(grow, 0, h / maps, 0);      // the head's output gate: sigmoid of its logit
   for (int d = threadIdx.x; d < dv; d += blockDim.x) {
     float acc = 0.f;
     for (int w2 = 0; w2 < NW; ++w2)
       if (wm[w2] != -INFINITY) acc = fmaf(wo[w2 * dv + d], expf(wm[w2] - M), acc);
+    if (gate && gate_ch) acc *= gate_factor(grow, gate_ch, h / maps, d);
     out[((size_t)t * HV + h) * dv + d] = from_f32<TO>(acc * inv);
   }
 }
@@ -425,7 +544,7 @@ masked_attn_kernel(const float* __restrict__ q, TO* __restrict__ out, const T* _
 // A block = up to 32 (token, query head) rows of one key/value head and of one run of consecutive tokens (a tile of the
 // step's metadata); a page of 64 keys with their values is staged in shared memory as float32 once for all the rows.
 // A warp owns four rows, so a key element read from shared memory serves four multiply-adds; lanes own keys for the
-// scores and value dimensions for the weighted sum.  Row r sees key p iff first[r] <= p <= its own position.
+// scores and value dimensions for the weighted sum.  Row r sees key p iff p <= its own position and (first[r] <= p or p < keep).
 constexpr int TM_RW = 4, TM_WARPS = 8, TM_ROWS = TM_RW * TM_WARPS, TM_KEYS = PAGE;
 
 // PAGE rows of n values from global memory (row pitch `src_pitch`) into shared memory as float32 (row pitch `dst_pitch`); rows from
@@ -470,7 +589,7 @@ masked_attn_tiled_kernel(const float* __restrict__ q, TO* __restrict__ out, cons
                          const int32_t* __restrict__ page_table, int table_stride, int n_pages, const int32_t* __restrict__ tile_seq,
                          const int32_t* __restrict__ tile_tok0, const int32_t* __restrict__ tile_ntok, const int32_t* __restrict__ tile_pos0,
                          int H, int G, int dk, int dv, float scale, int mask, int mask_size, const float* __restrict__ sink,
-                         int n_splits, float* __restrict__ part, int maps, const float* __restrict__ gate, int ldg) {
+                         int n_splits, float* __restrict__ part, int maps, const float* __restrict__ gate, int ldg, int keep, int gate_ch) {
   extern __shared__ float tm_smem[];
   pdl_launch_dependents();
   pdl_wait();
@@ -516,13 +635,17 @@ masked_attn_tiled_kernel(const float* __restrict__ q, TO* __restrict__ out, cons
 #pragma unroll
     for (int c = 0; c < NC; ++c) acc[r][c] = 0.f;
   }
-  int kt_begin = first_key(first_pos, mask, mask_size) / PAGE, kt_end = last_pos / PAGE;
+  // the pages to visit: those of the kept keys that lie ahead of the window's first, then the window's
+  const int kt_window = first_key(first_pos, mask, mask_size) / PAGE, kt_kept = min(kt_window, (keep + PAGE - 1) / PAGE);
+  const int n_visit = kt_kept + last_pos / PAGE - kt_window + 1;
+  int v_begin = 0, v_end = n_visit;
   if (n_splits > 1) {
-    const int per = (kt_end - kt_begin + n_splits) / n_splits;
-    kt_begin += split * per;
-    kt_end = min(kt_end, kt_begin + per - 1);
+    const int per = (n_visit - 1 + n_splits) / n_splits;
+    v_begin = split * per;
+    v_end = min(n_visit, v_begin + per);
   }
-  for (int kt = kt_begin; kt <= kt_end; ++kt) {
+  for (int vi = v_begin; vi < v_end; ++vi) {
+    const int kt = vi < kt_kept ? vi : kt_window + vi - kt_kept;
     const int page = paged ? pages[kt] : 0;
     const bool held = !paged || (page >= 0 && page < n_pages);
     const size_t first_row = paged ? ((size_t)(held ? page : 0) * G + g) * PAGE : ((size_t)(tok0 - pos0 + kt * PAGE) * G + g);
@@ -537,7 +660,7 @@ masked_attn_tiled_kernel(const float* __restrict__ q, TO* __restrict__ out, cons
 #pragma unroll
     for (int r = 0; r < TM_RW; ++r)
       if (limit[r] >= first[r]) { any_hi = max(any_hi, limit[r]); any_lo = min(any_lo, first[r]); }
-    if (base > any_hi || base + TM_KEYS - 1 < any_lo) continue;     // none of this warp's rows sees any of these keys
+    if (base > any_hi || (base + TM_KEYS - 1 < any_lo && base >= keep)) continue;     // none of this warp's rows sees any of these keys
     const int i0 = base + lane, i1 = i0 + 32;
     float s0[TM_RW] = {}, s1[TM_RW] = {};
     const float* k0 = Ks + lane * ks;
@@ -555,8 +678,8 @@ masked_attn_tiled_kernel(const float* __restrict__ q, TO* __restrict__ out, cons
     float corr[TM_RW];
 #pragma unroll
     for (int r = 0; r < TM_RW; ++r) {
-      const float a = i0 >= first[r] && i0 <= limit[r] ? s0[r] * scale : -INFINITY;
-      const float b = i1 >= first[r] && i1 <= limit[r] ? s1[r] * scale : -INFINITY;
+      const float a = (i0 >= first[r] || i0 < keep) && i0 <= limit[r] ? s0[r] * scale : -INFINITY;
+      const float b = (i1 >= first[r] || i1 < keep) && i1 <= limit[r] ? s1[r] * scale : -INFINITY;
       const float mx = fmaxf(m[r], warp_max(fmaxf(a, b)));
       float p0 = 0.f, p1 = 0.f;
       corr[r] = 1.f;
@@ -614,11 +737,14 @@ masked_attn_tiled_kernel(const float* __restrict__ q, TO* __restrict__ out, cons
       lr = lr * fix + expf(sk - mx);
     }
     float inv = lr > 0.f ? fix / lr : 0.f;
-    if (gate) inv *= 1.0f / (1.0f + expf(-gate[(size_t)(tok0 + tok) * ldg + head]));      // the head's output gate
+    const float* grow = gate ? gate + (size_t)(tok0 + tok) * ldg : nullptr;
+    if (gate && !gate_ch) inv *= gate_factor(grow, 0, head, 0);      // the head's output gate
 #pragma unroll
     for (int c = 0; c < NC; ++c) {
       const int d = lane + 32 * c;
-      if (d < dv) out[((size_t)(tok0 + tok) * HV + head * maps + mp) * dv + d] = from_f32<TO>(acc[r][c] * inv);
+      if (d >= dv) continue;
+      const float f = gate && gate_ch ? inv * gate_factor(grow, gate_ch, head, d) : inv;
+      out[((size_t)(tok0 + tok) * HV + head * maps + mp) * dv + d] = from_f32<TO>(acc[r][c] * f);
     }
   }
 }
@@ -626,7 +752,7 @@ masked_attn_tiled_kernel(const float* __restrict__ q, TO* __restrict__ out, cons
 // out[t][h][:] from the splits' partial results [t][h][split][2 + dv]: maxima, denominators, weighted values; the sink joins here
 template <typename TO>
 __global__ void masked_attn_fold_kernel(const float* __restrict__ part, TO* __restrict__ out, const float* __restrict__ sink, int H, int dv,
-                                        int n_splits, const float* __restrict__ gate, int ldg, int maps) {
+                                        int n_splits, const float* __restrict__ gate, int ldg, int maps, int gate_ch) {
   pdl_launch_dependents();
   pdl_wait();
   const int t = blockIdx.x, h = blockIdx.y;
@@ -639,13 +765,15 @@ __global__ void masked_attn_fold_kernel(const float* __restrict__ part, TO* __re
     if (ms != -INFINITY) L += p[(size_t)s * (2 + dv) + 1] * expf(ms - M);
   }
   float inv = L > 0.f ? 1.0f / L : 0.f;
-  if (gate) inv *= 1.0f / (1.0f + expf(-gate[(size_t)t * ldg + h / maps]));      // the head's output gate
+  const float* grow = gate ? gate + (size_t)t * ldg : nullptr;
+  if (gate && !gate_ch) inv *= gate_factor(grow, 0, h / maps, 0);      // the head's output gate
   for (int d = threadIdx.x; d < dv; d += blockDim.x) {
     float acc = 0.f;
     for (int s = 0; s < n_splits; ++s) {
       const float ms = p[(size_t)s * (2 + dv)];
       if (ms != -INFINITY) acc = fmaf(p[(size_t)s * (2 + dv) + 2 + d], expf(ms - M), acc);
     }
+    if (gate && gate_ch) acc *= gate_factor(grow, gate_ch, h / maps, d);
     out[((size_t)t * H + h) * dv + d] = from_f32<TO>(acc * inv);
   }
 }
@@ -724,24 +852,70 @@ extern "C" int edgelm_rotate_append(const float* qkv, const float* bias, float* 
   return 0;
 }
 
+// `rotate_append` with the norm over the whole projection (see `norm_append_kernel`)
+extern "C" int edgelm_norm_append(const float* qkv, const float* bias, float* q_out, const int32_t* tok_pos, const int32_t* tok_seq,
+                                  const int32_t* page_table, int table_stride, int n_pages, void* kcache, void* vcache, int dtype, int n_tokens,
+                                  int H, int G, int dk, int dv, int rot, int interleaved, const double* freq, int* err, const float* q_norm,
+                                  const float* k_norm, float eps, int ldq, float mult, cudaStream_t stream) {
+  if (n_tokens == 0) return 0;
+  EL_REFUSE(n_tokens > 0 && H > 0 && G > 0 && H % G == 0 && dk >= 1 && dv >= 1, "norm_append: %d query heads over %d key/value heads of %d / %d", H, G, dk, dv);
+  EL_REFUSE(ldq >= (H + G) * dk + G * dv && q_norm != nullptr && k_norm != nullptr, "norm_append: rows of %d values do not hold the heads, or no weights", ldq);
+  EL_REFUSE(rot >= 0 && rot <= dk && rot % 2 == 0 && (rot == 0 || freq != nullptr), "norm_append: %d rotated dimensions of %d", rot, dk);
+  const size_t smem = (size_t)(H + G) * dk * sizeof(float);
+  EL_REFUSE(smem <= 200 * 1024, "norm_append: a row of %d query and key values is too long", (H + G) * dk);
+  const bool vec = dk % 4 == 0 && dv % 4 == 0 && ldq % 4 == 0 && (uintptr_t)qkv % 16 == 0 && (uintptr_t)q_out % 16 == 0 &&
+                   (uintptr_t)kcache % 16 == 0 && (uintptr_t)vcache % 16 == 0;
+  // (few tokens: as many threads as the row has pieces, so that a row is a trip or two to memory)
+  const int pieces = (H + G) * dk / (vec ? 4 : 1), most = n_tokens <= 64 ? 1024 : 256;
+  int threads = 128;
+  while (threads < most && threads < pieces) threads *= 2;
+  const int bit = pdl_bit_for_tokens(n_tokens);
+#define EL_NA(T, V) do { auto kern = norm_append_kernel<T, V>; \
+    if (smem > 48 * 1024) cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
+    launch_pdl(bit, kern, dim3(n_tokens), dim3(threads), smem, stream, qkv, bias, q_out, tok_pos, tok_seq, page_table, table_stride, n_pages, (T*)kcache, \
+               (T*)vcache, H, G, dk, dv, rot, interleaved, freq, err, q_norm, k_norm, eps, ldq, mult); } while (0)
+  if (dtype == DT_F32) { if (vec) EL_NA(float, 4); else EL_NA(float, 1); }
+  else if (dtype == DT_BF16) { if (vec) EL_NA(__nv_bfloat16, 4); else EL_NA(__nv_bfloat16, 1); }
+  else EL_REFUSE(false, "norm_append: unknown dtype code %d", dtype);
+#undef EL_NA
+  EL_LAUNCH_CHECK("norm_append");
+  return 0;
+}
+
+// rows[t][0 .. n) = the cache row of token t, one key head of n values
+extern "C" int edgelm_latent_rows(const void* kcache, void* rows, int dtype, const int32_t* tok_pos, const int32_t* tok_seq,
+                                  const int32_t* page_table, int table_stride, int n_pages, int n, int n_tokens, int* err, cudaStream_t stream) {
+  if (n_tokens == 0) return 0;
+  EL_REFUSE(n_tokens > 0 && n >= 1, "latent_rows: bad sizes");
+  const dim3 grid((n_tokens + 3) / 4), block(64, 4);
+  const int bit = pdl_bit_for_tokens(n_tokens);
+  if (dtype == DT_F32) launch_pdl(bit, latent_rows_kernel<float>, grid, block, (size_t)0, stream, (const float*)kcache, (float*)rows, tok_pos, tok_seq, page_table, table_stride, n_pages, n, n_tokens, err);
+  else if (dtype == DT_BF16) launch_pdl(bit, latent_rows_kernel<__nv_bfloat16>, grid, block, (size_t)0, stream, (const __nv_bfloat16*)kcache, (__nv_bfloat16*)rows, tok_pos, tok_seq, page_table, table_stride, n_pages, n, n_tokens, err);
+  else EL_REFUSE(false, "latent_rows: unknown dtype code %d", dtype);
+  EL_LAUNCH_CHECK("latent_rows");
+  return 0;
+}
+
 extern "C" int edgelm_latent_prepare(const float* u, int ldu, int kv_off, int has_kv, float* q_out, int q_pitch, int q_off, int copy_q,
                                      const float* norm_w, float eps, const int32_t* tok_pos, const int32_t* tok_seq,
                                      const int32_t* page_table, int table_stride, int n_pages, void* kcache, void* row_out, int dtype,
                                      int n_tokens, int H, int d, int rd, int r, const double* freq, int* err, int interleaved, float mult,
-                                     cudaStream_t stream) {
+                                     int ql_off, int ql_rank, const float* ql_w, void* ql_out, cudaStream_t stream) {
   if (n_tokens == 0) return 0;
-  EL_REFUSE(n_tokens > 0 && H > 0 && d >= 0 && r >= 1 && rd >= 0 && rd % 2 == 0, "latent_prepare: sizes heads %d, %d + %d, latent %d", H, d, rd, r);
+  EL_REFUSE(ql_out == nullptr || (ql_rank >= 1 && ql_off >= 0 && ql_off + ql_rank <= ldu && ql_w != nullptr), "latent_prepare: a query latent of %d from column %d", ql_rank, ql_off);
+  EL_REFUSE(n_tokens > 0 && H >= 0 && d >= 0 && r >= 1 && rd >= 0 && rd % 2 == 0, "latent_prepare: sizes heads %d, %d + %d, latent %d", H, d, rd, r);
   EL_REFUSE(rd == 0 || freq != nullptr, "latent_prepare: no frequencies");
   EL_REFUSE(H * (d + rd) <= ldu && (!has_kv || kv_off + r + rd <= ldu), "latent_prepare: rows of %d values are too short", ldu);
-  EL_REFUSE(q_off >= (copy_q ? d : 0) && q_off + rd <= q_pitch, "latent_prepare: a query head of %d values does not hold %d at %d", q_pitch, rd, q_off);
+  EL_REFUSE(H == 0 || (q_off >= (copy_q ? d : 0) && q_off + rd <= q_pitch), "latent_prepare: a query head of %d values does not hold %d at %d", q_pitch, rd, q_off);
   const int bit = pdl_bit_for_tokens(n_tokens);
   if (dtype == DT_F32)
     launch_pdl(bit, latent_prepare_kernel<float>, dim3(n_tokens), dim3(256), (size_t)0, stream, u, ldu, kv_off, has_kv, q_out, q_pitch, q_off, copy_q,
-               norm_w, eps, tok_pos, tok_seq, page_table, table_stride, n_pages, (float*)kcache, (float*)row_out, H, d, rd, r, freq, err, interleaved, mult);
+               norm_w, eps, tok_pos, tok_seq, page_table, table_stride, n_pages, (float*)kcache, (float*)row_out, H, d, rd, r, freq, err, interleaved, mult,
+               ql_off, ql_rank, ql_w, (float*)ql_out);
   else if (dtype == DT_BF16)
     launch_pdl(bit, latent_prepare_kernel<__nv_bfloat16>, dim3(n_tokens), dim3(256), (size_t)0, stream, u, ldu, kv_off, has_kv, q_out, q_pitch, q_off,
                copy_q, norm_w, eps, tok_pos, tok_seq, page_table, table_stride, n_pages, (__nv_bfloat16*)kcache, (__nv_bfloat16*)row_out, H, d, rd,
-               r, freq, err, interleaved, mult);
+               r, freq, err, interleaved, mult, ql_off, ql_rank, ql_w, (__nv_bfloat16*)ql_out);
   else
     EL_REFUSE(false, "latent_prepare: unknown dtype code %d", dtype);
   EL_LAUNCH_CHECK("latent_prepare");
@@ -789,7 +963,9 @@ extern "C" int edgelm_add_row_bias(float* x, const float* b, int n_tokens, int d
   return 0;
 }
 
-static int masked_common_check(const char* what, int H, int G, int dk, int dv, int mask, int mask_size, int dtype, int out_dtype) {
+static int masked_common_check(const char* what, int H, int G, int dk, int dv, int mask, int mask_size, int dtype, int out_dtype, int keep, int gate_ch, int maps) {
+  EL_REFUSE(keep >= 0 && (keep == 0 || mask == MASK_WINDOW), "%s: %d kept keys without a window", what, keep);
+  EL_REFUSE(gate_ch == 0 || (gate_ch == dv && maps == 1), "%s: a gate of %d channels over values of %d and %d maps", what, gate_ch, dv, maps);
   EL_REFUSE(H > 0 && G > 0 && H % G == 0, "%s: %d query heads over %d key/value heads", what, H, G);
   EL_REFUSE(dk >= 1 && dk <= 1024 && dv >= 1 && dv <= 512, "%s: head sizes %d / %d are not taken (keys to 1024, values to 512)", what, dk, dv);
   EL_REFUSE(mask == MASK_CAUSAL || ((mask == MASK_WINDOW || mask == MASK_CHUNK) && mask_size >= 1), "%s: mask %d of size %d", what, mask, mask_size);
@@ -802,7 +978,7 @@ template <typename T, typename TO, int DVR>
 static void launch_masked(const float* q, void* out, const void* kcache, const void* vcache, const int32_t* tok_pos, const int32_t* tok_seq,
                           const int32_t* page_table, int table_stride, int n_pages, int n_tokens, int H, int G, int dk, int dv, float scale,
                           int mask, int mask_size, const float* sink, int warps, int maps, const float* gate, int ldg, int n_splits, float* part,
-                          cudaStream_t stream) {
+                          int keep, int gate_ch, cudaStream_t stream) {
   const T* vb = vcache ? (const T*)vcache : (const T*)kcache;
   const int ldv = vcache ? dv : dk;
   const int vec_k = (dk % (16 / (int)sizeof(T)) == 0) && ((uintptr_t)kcache % 16 == 0);
@@ -810,28 +986,30 @@ static void launch_masked(const float* q, void* out, const void* kcache, const v
   auto kern = masked_attn_kernel<T, TO, DVR>;
   if (smem > 48 * 1024) cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
   launch_pdl(pdl_bit_for_tokens(n_tokens), kern, dim3(n_tokens, H * maps, n_splits), dim3(warps * 32), smem, stream, q, (TO*)out, (const T*)kcache, vb, ldv,
-             tok_pos, tok_seq, page_table, table_stride, n_pages, H, G, dk, dv, scale, mask, mask_size, sink, vec_k, maps, gate, ldg, n_splits, part);
+             tok_pos, tok_seq, page_table, table_stride, n_pages, H, G, dk, dv, scale, mask, mask_size, sink, vec_k, maps, gate, ldg, n_splits, part, keep, gate_ch);
   if (n_splits > 1 && cudaPeekAtLastError() == cudaSuccess)
     launch_pdl(pdl_bit_for_tokens(n_tokens), masked_attn_fold_kernel<TO>, dim3(n_tokens, H * maps), dim3(dv >= 256 ? 256 : 128), (size_t)0, stream,
-               (const float*)part, (TO*)out, sink, H * maps, dv, n_splits, gate, ldg, maps);
+               (const float*)part, (TO*)out, sink, H * maps, dv, n_splits, gate, ldg, maps, gate_ch);
 }
 
 // `vcache` null: the values are the first dv dimensions of the key rows.  `max_keys`: the most keys a token of the step sees
 // (chooses how many warps share a token's keys).  `n_splits` > 1: a token's keys are dealt to so many blocks, whose partial
 // results go through `part` (n_tokens H maps n_splits (2 + dv) floats) and are merged by a second launch.  `maps` > 1: every query head and key row holds `maps` runs of dk dimensions,
-// each an attention of its own over the head's values; q [tokens][H][maps][dk], out [tokens][H][maps][dv].
+// each an attention of its own over the head's values; q [tokens][H][maps][dk], out [tokens][H][maps][dv].  `keep`: with a window,
+// the sequence's first keys that stay visible.  `gate_ch`: 0, a gate number per head; dv, one per channel.
 extern "C" int edgelm_masked_attn(const float* q, void* out, int out_dtype, const void* kcache, const void* vcache, int dtype,
                                   const int32_t* tok_pos, const int32_t* tok_seq, const int32_t* page_table, int table_stride, int n_pages,
                                   int n_tokens, int H, int G, int dk, int dv, float scale, int mask, int mask_size, const float* sink,
-                                  int max_keys, int maps, const float* gate, int ldg, int n_splits, float* part, cudaStream_t stream) {
+                                  int max_keys, int maps, const float* gate, int ldg, int n_splits, float* part, int keep, int gate_ch,
+                                  cudaStream_t stream) {
   if (n_tokens == 0) return 0;
   EL_REFUSE(n_splits >= 1 && n_splits <= 64 && (n_splits == 1 || part != nullptr), "masked_attn: %d splits", n_splits);
   if (n_splits > 1) max_keys = (max_keys + n_splits - 1) / n_splits;
-  if (masked_common_check("masked_attn", H, G, dk, dv, mask, mask_size, dtype, out_dtype)) return -1;
+  if (masked_common_check("masked_attn", H, G, dk, dv, mask, mask_size, dtype, out_dtype, keep, gate_ch, maps)) return -1;
   EL_REFUSE(maps >= 1 && H * maps <= 65535 && (maps == 1 || (sink == nullptr && vcache != nullptr)), "masked_attn: %d maps take no sink and values of their own", maps);
   EL_REFUSE(vcache != nullptr || dv <= dk, "masked_attn: values of %d inside keys of %d", dv, dk);
   const int warps = max_keys <= 64 ? 2 : (max_keys <= 256 ? 4 : MA_MAX_WARPS);
-#define EL_MA2(T, TO, DVR) launch_masked<T, TO, DVR>(q, out, kcache, vcache, tok_pos, tok_seq, page_table, table_stride, n_pages, n_tokens, H, G, dk, dv, scale, mask, mask_size, sink, warps, maps, gate, ldg, n_splits, part, stream)
+#define EL_MA2(T, TO, DVR) launch_masked<T, TO, DVR>(q, out, kcache, vcache, tok_pos, tok_seq, page_table, table_stride, n_pages, n_tokens, H, G, dk, dv, scale, mask, mask_size, sink, warps, maps, gate, ldg, n_splits, part, keep, gate_ch, stream)
 #define EL_MA(DVR) do { if (dtype == DT_F32) EL_MA2(float, float, DVR); else if (out_dtype == DT_F32) EL_MA2(__nv_bfloat16, float, DVR); else EL_MA2(__nv_bfloat16, __nv_bfloat16, DVR); } while (0)
   if (dv <= 32) EL_MA(1); else if (dv <= 64) EL_MA(2); else if (dv <= 128) EL_MA(4); else if (dv <= 256) EL_MA(8); else EL_MA(16);
 #undef EL_MA
@@ -855,8 +1033,8 @@ template <typename T, typename TO, int NC>
 static int launch_masked_tiled(const float* q, void* out, const void* kcache, const void* vcache, const int32_t* page_table, int table_stride,
                                int n_pages, const int32_t* tile_seq, const int32_t* tile_tok0, const int32_t* tile_ntok, const int32_t* tile_pos0,
                                int n_tiles, int max_tile_tokens, int H, int G, int dk, int dv, float scale, int mask, int mask_size,
-                               const float* sink, int n_splits, float* part, int n_tokens, int maps, const float* gate, int ldg,
-                               cudaStream_t stream) {
+                               const float* sink, int n_splits, float* part, int n_tokens, int maps, const float* gate, int ldg, int keep,
+                               int gate_ch, cudaStream_t stream) {
   const size_t smem = tiled_smem(dk, dv, vcache != nullptr);
   EL_REFUSE(smem <= TM_MAX_SMEM, "masked_attn_tiled: heads of %d / %d need %zu bytes of shared memory", dk, dv, smem);
   auto kern = masked_attn_tiled_kernel<T, TO, NC>;
@@ -865,11 +1043,11 @@ static int launch_masked_tiled(const float* q, void* out, const void* kcache, co
   const dim3 grid(n_tiles, G * maps, ((max_tile_tokens * grp + TM_ROWS - 1) / TM_ROWS) * n_splits);
   const int bit = pdl_bit_for_tokens(n_tokens);
   launch_pdl(bit, kern, grid, dim3(TM_WARPS * 32), smem, stream, q, (TO*)out, (const T*)kcache, (const T*)vcache, page_table, table_stride, n_pages,
-             tile_seq, tile_tok0, tile_ntok, tile_pos0, H, G, dk, dv, scale, mask, mask_size, sink, n_splits, part, maps, gate, ldg);
+             tile_seq, tile_tok0, tile_ntok, tile_pos0, H, G, dk, dv, scale, mask, mask_size, sink, n_splits, part, maps, gate, ldg, keep, gate_ch);
   if (n_splits > 1) {
     if (cudaGetLastError() != cudaSuccess) return 0;   // (the caller reports it)
     launch_pdl(bit, masked_attn_fold_kernel<TO>, dim3(n_tokens, H * maps), dim3(dv >= 256 ? 256 : 128), (size_t)0, stream, (const float*)part, (TO*)out, sink,
-               H * maps, dv, n_splits, gate, ldg, maps);
+               H * maps, dv, n_splits, gate, ldg, maps, gate_ch);
   }
   return 0;
 }
@@ -878,16 +1056,16 @@ extern "C" int edgelm_masked_attn_tiled(const float* q, void* out, int out_dtype
                                         const int32_t* page_table, int table_stride, int n_pages, const int32_t* tile_seq,
                                         const int32_t* tile_tok0, const int32_t* tile_ntok, const int32_t* tile_pos0, int n_tiles,
                                         int max_tile_tokens, int H, int G, int dk, int dv, float scale, int mask, int mask_size,
-                                        const float* sink, int n_splits, float* part, int n_tokens, int maps, const float* gate, int ldg,
-                                        cudaStream_t stream) {
+                                        const float* sink, int n_splits, float* part, int n_tokens, int maps, const float* gate, int ldg, int keep,
+                                        int gate_ch, cudaStream_t stream) {
   if (n_tiles == 0) return 0;
   EL_REFUSE(maps >= 1 && G * maps <= 65535 && (maps == 1 || (sink == nullptr && vcache != nullptr)), "masked_attn_tiled: %d maps take no sink and values of their own", maps);
   EL_REFUSE(n_splits >= 1 && n_splits <= 64 && (n_splits == 1 || part != nullptr) && n_tokens > 0, "masked_attn_tiled: %d splits", n_splits);
-  if (masked_common_check("masked_attn_tiled", H, G, dk, dv, mask, mask_size, dtype, out_dtype)) return -1;
+  if (masked_common_check("masked_attn_tiled", H, G, dk, dv, mask, mask_size, dtype, out_dtype, keep, gate_ch, maps)) return -1;
   EL_REFUSE(n_tiles > 0 && max_tile_tokens > 0 && G <= 65535, "masked_attn_tiled: bad tile counts");
   EL_REFUSE(vcache != nullptr || dv <= dk, "masked_attn_tiled: values of %d inside keys of %d", dv, dk);
   int rc = 0;
-#define EL_MT2(T, TO, NC) rc = launch_masked_tiled<T, TO, NC>(q, out, kcache, vcache, page_table, table_stride, n_pages, tile_seq, tile_tok0, tile_ntok, tile_pos0, n_tiles, max_tile_tokens, H, G, dk, dv, scale, mask, mask_size, sink, n_splits, part, n_tokens, maps, gate, ldg, stream)
+#define EL_MT2(T, TO, NC) rc = launch_masked_tiled<T, TO, NC>(q, out, kcache, vcache, page_table, table_stride, n_pages, tile_seq, tile_tok0, tile_ntok, tile_pos0, n_tiles, max_tile_tokens, H, G, dk, dv, scale, mask, mask_size, sink, n_splits, part, n_tokens, maps, gate, ldg, keep, gate_ch, stream)
 #define EL_MT(NC) do { if (dtype == DT_F32) EL_MT2(float, float, NC); else if (out_dtype == DT_F32) EL_MT2(__nv_bfloat16, float, NC); else EL_MT2(__nv_bfloat16, __nv_bfloat16, NC); } while (0)
   if (dv <= 32) EL_MT(1); else if (dv <= 64) EL_MT(2); else if (dv <= 128) EL_MT(4); else if (dv <= 256) EL_MT(8); else EL_MT(16);
 #undef EL_MT

@@ -16,7 +16,8 @@
 // barrier of its own; the groups' partial (maximum, sum, output) are merged in shared memory in the order of the groups.
 // An optional gate per (token, head) multiplies the head's output by its sigmoid before the rounding; an optional sink per head is
 // one more term exp(sink_h) of the softmax's denominator, without a key, a value or the scale.
-// Masks as in the CUDA-core kernels: causal, a sliding window, or chunks; pages before the first key that the tile's first row sees
+// (or, with a gate per channel, every channel by its own).
+// Masks as in the CUDA-core kernels: causal, a sliding window (with the sequence's first `keep` keys kept visible), or chunks; pages before the first key that the tile's first row sees
 // are not visited.  Keys and values come from the cache's pages (the page table's rows are the step's sequences) or, without a page
 // table, from the step's own rows (every sequence of the step then starts at position 0).
 // Takes key head sizes 32, 64, 96, 128 over value head sizes of these that are not larger.
@@ -76,7 +77,7 @@ attn_prefill_split_kernel(const float* __restrict__ q, int ldq, __nv_bfloat16* _
                           const int32_t* __restrict__ page_table, int table_stride, const int32_t* __restrict__ tile_seq,
                           const int32_t* __restrict__ tile_tok0, const int32_t* __restrict__ tile_ntok,
                           const int32_t* __restrict__ tile_pos0, int nh, int nkv, float scale, const float* __restrict__ gate, int ldg,
-                          int mask, int mask_size, const float* __restrict__ sink) {
+                          int mask, int mask_size, const float* __restrict__ sink, int keep, int gate_ch) {
   constexpr int HD = HDT * 16, VD = VDT * 16;
   constexpr int PITCH = HD + 8, VPITCH = VD + 8;   // elements: 16 bytes of padding per row
   constexpr int CHUNKS = HD / 8, VCHUNKS = VD / 8; // 16-byte chunks per row
@@ -100,7 +101,10 @@ attn_prefill_split_kernel(const float* __restrict__ q, int ldq, __nv_bfloat16* _
   // what the mask leaves out in front: per row, and for the warp's first (the smallest) and last row
   const int firstA = sp_first_key(max(limA, 0), mask, mask_size), firstB = sp_first_key(max(limB, 0), mask, mask_size);
   const int warp_first = sp_first_key(max(warp_min_limit, 0), mask, mask_size), warp_last_first = sp_first_key(max(warp_limit, 0), mask, mask_size);
-  const int first_page = sp_first_key(pos0, mask, mask_size) / PAGE;
+  // the pages to visit: those of the kept keys that lie ahead of the window's first, then the window's
+  const int first_page = sp_first_key(pos0, mask, mask_size) / PAGE, kept_pages = min(first_page, (keep + PAGE - 1) / PAGE);
+  const int n_visit = kept_pages + n_pages - first_page;
+  auto page_at = [&](int i) { return i < kept_pages ? i : first_page + i - kept_pages; };
   const float scale2 = scale * 1.4426950408889634f;                     // scores in units of log 2
 
   auto load_page = [&](int pg, int stage) {
@@ -155,17 +159,17 @@ attn_prefill_split_kernel(const float* __restrict__ q, int ldq, __nv_bfloat16* _
     if (NG == 1) __syncthreads();
     else asm volatile("bar.sync %0, %1;" ::"r"(group + 1), "r"(SP_WARPS * 32) : "memory");
   };
-  if (first_page + group < n_pages) load_page(first_page + group, 0);
-  for (int pg = first_page + group, it = 0; pg < n_pages; pg += NG, ++it) {
-    const int stage = it & 1;
-    if (pg + NG < n_pages) {
-      load_page(pg + NG, stage ^ 1);
+  if (group < n_visit) load_page(page_at(group), 0);
+  for (int vi = group, it = 0; vi < n_visit; vi += NG, ++it) {
+    const int stage = it & 1, pg = page_at(vi);
+    if (vi + NG < n_visit) {
+      load_page(page_at(vi + NG), stage ^ 1);
       asm volatile("cp.async.wait_group 1;" ::: "memory");
     } else {
       asm volatile("cp.async.wait_group 0;" ::: "memory");
     }
     group_sync();
-    if (pg * PAGE <= warp_limit && pg * PAGE + PAGE - 1 >= warp_first) {   // else: no row of this warp sees this page
+    if (pg * PAGE <= warp_limit && (pg * PAGE + PAGE - 1 >= warp_first || pg * PAGE < keep)) {   // else: no row of this warp sees this page
       const __nv_bfloat16* ks = sm + stage * STAGE;
       const __nv_bfloat16* vs = ks + PAGE * PITCH;
       // ---- S = Q K^T : 8 tiles of 8 keys, three query terms against every key fragment
@@ -188,16 +192,16 @@ attn_prefill_split_kernel(const float* __restrict__ q, int ldq, __nv_bfloat16* _
         }
       }
       // ---- scale, mask, running max and sum (float32), scores in units of log 2
-      const bool masked = pg * PAGE + PAGE - 1 > warp_min_limit || pg * PAGE < warp_last_first;
+      const bool masked = pg * PAGE + PAGE - 1 > warp_min_limit || (pg * PAGE < warp_last_first && pg * PAGE + PAGE > keep);
       float mxA = -CUDART_INF_F, mxB = -CUDART_INF_F;
 #pragma unroll
       for (int nt = 0; nt < 8; ++nt) {
         const int key = pg * PAGE + nt * 8 + tig * 2;
         if (masked) {
-          s[nt][0] = key >= firstA && key <= limA ? s[nt][0] * scale2 : -CUDART_INF_F;
-          s[nt][1] = key + 1 >= firstA && key + 1 <= limA ? s[nt][1] * scale2 : -CUDART_INF_F;
-          s[nt][2] = key >= firstB && key <= limB ? s[nt][2] * scale2 : -CUDART_INF_F;
-          s[nt][3] = key + 1 >= firstB && key + 1 <= limB ? s[nt][3] * scale2 : -CUDART_INF_F;
+          s[nt][0] = (key >= firstA || key < keep) && key <= limA ? s[nt][0] * scale2 : -CUDART_INF_F;
+          s[nt][1] = (key + 1 >= firstA || key + 1 < keep) && key + 1 <= limA ? s[nt][1] * scale2 : -CUDART_INF_F;
+          s[nt][2] = (key >= firstB || key < keep) && key <= limB ? s[nt][2] * scale2 : -CUDART_INF_F;
+          s[nt][3] = (key + 1 >= firstB || key + 1 < keep) && key + 1 <= limB ? s[nt][3] * scale2 : -CUDART_INF_F;
         } else {
           s[nt][0] *= scale2;
           s[nt][1] *= scale2;
@@ -318,13 +322,25 @@ attn_prefill_split_kernel(const float* __restrict__ q, int ldq, __nv_bfloat16* _
     lB = lB * fixB + exp2f(s2 - nmB);
   }
   float invA = lA > 0.f ? fixA / lA : 0.f, invB = lB > 0.f ? fixB / lB : 0.f;
-  if (gate != nullptr) {      // the head's output gate: sigmoid of its logit
+  if (gate != nullptr && !gate_ch) {      // the head's output gate: sigmoid of its logit
     if (rowA < ntok) invA *= 1.0f / (1.0f + expf(-gate[(size_t)(tok0 + rowA) * ldg + head]));
     if (rowB < ntok) invB *= 1.0f / (1.0f + expf(-gate[(size_t)(tok0 + rowB) * ldg + head]));
   }
 #pragma unroll
   for (int dt = 0; dt < VD / 8; ++dt) {
     const int d = head * VD + dt * 8 + tig * 2;
+    if (gate != nullptr && gate_ch) {     // a gate per channel
+      if (rowA < ntok) {
+        const float* ga = gate + (size_t)(tok0 + rowA) * ldg + d;
+        o[dt][0] *= 1.0f / (1.0f + expf(-ga[0]));
+        o[dt][1] *= 1.0f / (1.0f + expf(-ga[1]));
+      }
+      if (rowB < ntok) {
+        const float* gb = gate + (size_t)(tok0 + rowB) * ldg + d;
+        o[dt][2] *= 1.0f / (1.0f + expf(-gb[0]));
+        o[dt][3] *= 1.0f / (1.0f + expf(-gb[1]));
+      }
+    }
     if (rowA < ntok) {
       const __nv_bfloat162 v = __floats2bfloat162_rn(o[dt][0] * invA, o[dt][1] * invA);
       *reinterpret_cast<__nv_bfloat162*>(out + (size_t)(tok0 + rowA) * ldo + d) = v;
@@ -350,6 +366,7 @@ struct SplitArgs {
   const float* gate;
   int ldg, mask, mask_size;
   const float* sink;
+  int keep, gate_ch;
 };
 
 template <int HDT, int VDT, int NG>
@@ -365,7 +382,7 @@ static int launch_split_ng(const SplitArgs& a, cudaStream_t stream) {
   }
   kern<<<dim3(a.n_tiles, a.nh), SP_WARPS * 32 * NG, smem, stream>>>(a.q, a.ldq, (__nv_bfloat16*)a.out, a.ldo, (const __nv_bfloat16*)a.kc, (const __nv_bfloat16*)a.vc,
                                                                      a.page_table, a.table_stride, a.tile_seq, a.tile_tok0, a.tile_ntok, a.tile_pos0, a.nh, a.nkv,
-                                                                     a.scale, a.gate, a.ldg, a.mask, a.mask_size, a.sink);
+                                                                     a.scale, a.gate, a.ldg, a.mask, a.mask_size, a.sink, a.keep, a.gate_ch);
   return 0;
 }
 
@@ -390,25 +407,27 @@ extern "C" int edgelm_attn_prefill_split_takes(int dk, int dv) { return split_si
 // pages [page][kv head][64][dk or dv] with `page_table` rows for the step's sequences (tile_seq indexes them), or, with `page_table`
 // null, the step's own rows [token][kv head][dk or dv] (every sequence of the step starts at position 0); tiles of at most 64 new
 // tokens of one sequence each.  `mask` 0 causal, 1 a window of `mask_size` keys, 2 chunks of `mask_size` positions.  `sink` (or
-// null): float32 [nh].  `gate` (or null): float32 [tokens][>= nh] with row pitch ldg.  `max_keys`: the most keys a tile attends over
+// null): float32 [nh].  `keep`: with a window, the sequence's first keys that stay visible.  `gate` (or null): float32 with row pitch
+// ldg, a number per head (`gate_ch` 0) or per channel (`gate_ch` = dv).  `max_keys`: the most keys a tile attends over
 // (a hint for how many warp groups share a tile's pages).
 extern "C" int edgelm_attn_prefill_split(const float* q, int ldq, void* out, int ldo, const void* kcache, const void* vcache,
                                          const int32_t* page_table, int table_stride, const int32_t* tile_seq, const int32_t* tile_tok0,
                                          const int32_t* tile_ntok, const int32_t* tile_pos0, int n_tiles, int nh, int nkv, int dk, int dv,
                                          float scale, int mask, int mask_size, const float* sink, const float* gate, int ldg, int max_keys,
-                                         cudaStream_t stream) {
+                                         int keep, int gate_ch, cudaStream_t stream) {
   if (n_tiles == 0) return 0;
   EL_REFUSE(nh > 0 && nkv > 0 && nh % nkv == 0, "attn_prefill_split: %d query heads are not a multiple of %d key/value heads", nh, nkv);
   EL_REFUSE(edgelm_attn_prefill_split_takes(dk, dv), "attn_prefill_split: head sizes %d / %d (takes 32, 64, 96, 128, values not larger than keys)", dk, dv);
   EL_REFUSE(ldq % 2 == 0 && ldo % 2 == 0 && (uintptr_t)q % 8 == 0 && (uintptr_t)out % 4 == 0, "attn_prefill_split: rows must be 8- and 4-byte aligned");
   EL_REFUSE((uintptr_t)kcache % 16 == 0 && (uintptr_t)vcache % 16 == 0, "attn_prefill_split: keys and values must be 16-byte aligned");
   EL_REFUSE(mask == SP_MASK_CAUSAL || ((mask == SP_MASK_WINDOW || mask == SP_MASK_CHUNK) && mask_size >= 1), "attn_prefill_split: mask %d of size %d", mask, mask_size);
+  EL_REFUSE(keep >= 0 && (keep == 0 || mask == SP_MASK_WINDOW) && (gate_ch == 0 || gate_ch == dv), "attn_prefill_split: %d kept keys, a gate of %d channels", keep, gate_ch);
   EL_REFUSE(n_tiles > 0 && nh <= 65535, "attn_prefill_split: bad grid");
   const long long blocks = (long long)n_tiles * nh;
-  if (mask != SP_MASK_CAUSAL && max_keys > mask_size + SP_ROWS) max_keys = mask_size + SP_ROWS;
+  if (mask != SP_MASK_CAUSAL && max_keys > mask_size + keep + SP_ROWS) max_keys = mask_size + keep + SP_ROWS;
   const int groups = ((max_keys + PAGE - 1) / PAGE >= 6 && blocks < 4 * 148 * 2) ? 2 : 1;
   const SplitArgs a{q, ldq, out, ldo, kcache, vcache, page_table, table_stride, tile_seq, tile_tok0, tile_ntok, tile_pos0, n_tiles, nh, nkv, scale,
-                    gate, ldg, mask, mask_size, sink};
+                    gate, ldg, mask, mask_size, sink, keep, gate_ch};
   int rc = 0;
 #define EL_SP(H, V) case (H) * 16 + (V): rc = launch_split<H, V>(groups, a, stream); break;
   switch (dk / 16 * 16 + dv / 16) {

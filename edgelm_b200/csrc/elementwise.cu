@@ -146,6 +146,24 @@ __global__ void rmsnorm_pair_kernel(float* __restrict__ x, const float* __restri
   }
 }
 
+// out[t][j] = gelu_tanh(u[t][j]) * table[ids[t]][j]: a row of numbers of a token's own, gated by the stream (u: a projection of it)
+template <typename T>
+__global__ void token_gate_kernel(const float* __restrict__ u, const int32_t* __restrict__ ids, const T* __restrict__ table, T* __restrict__ out,
+                                  int n_tokens, int dim, int vocab, int* __restrict__ err) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int i = blockIdx.x * blockDim.x + threadIdx.x;
+  if (i >= n_tokens * dim) return;
+  const int t = i / dim, j = i - t * dim, id = ids[t];
+  if (id < 0 || id >= vocab) {
+    if (j == 0) atomicOr(err, ERR_TOKEN_RANGE);
+    out[i] = from_f32<T>(0.f);
+    return;
+  }
+  const float z = u[i];
+  out[i] = from_f32<T>(0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z))) * to_f32(table[(size_t)id * dim + j]));
+}
+
 // z <- cap * tanh(z / cap), in place
 __global__ void softcap_kernel(float* __restrict__ z, size_t n, float cap) {
   pdl_launch_dependents();
@@ -311,6 +329,19 @@ extern "C" int edgelm_rmsnorm_pair(float* x, const float* add, const float* w1, 
   else if (out_dtype == DT_BF16) launch_pdl(32, rmsnorm_pair_kernel<__nv_bfloat16>, grid, block, (size_t)0, stream, x, add, w1, w2, (__nv_bfloat16*)y1, (__nv_bfloat16*)y2, dim, eps);
   else EL_REFUSE(false, "rmsnorm_pair: unknown dtype code %d", out_dtype);
   EL_LAUNCH_CHECK("rmsnorm_pair");
+  return 0;
+}
+
+extern "C" int edgelm_token_gate(const float* u, const int32_t* ids, const void* table, void* out, int dtype, int n_tokens, int dim, int vocab,
+                                 int* err, cudaStream_t stream) {
+  if (n_tokens == 0) return 0;
+  EL_REFUSE(n_tokens > 0 && dim > 0 && vocab > 0 && (long long)n_tokens * dim < (1LL << 31), "token_gate: bad sizes tokens=%d dim=%d vocab=%d", n_tokens, dim, vocab);
+  const dim3 grid((n_tokens * dim + 255) / 256), block(256);
+  const int bit = pdl_bit_for_tokens(n_tokens);
+  if (dtype == DT_F32) launch_pdl(bit, token_gate_kernel<float>, grid, block, (size_t)0, stream, u, ids, (const float*)table, (float*)out, n_tokens, dim, vocab, err);
+  else if (dtype == DT_BF16) launch_pdl(bit, token_gate_kernel<__nv_bfloat16>, grid, block, (size_t)0, stream, u, ids, (const __nv_bfloat16*)table, (__nv_bfloat16*)out, n_tokens, dim, vocab, err);
+  else EL_REFUSE(false, "token_gate: unknown dtype code %d", dtype);
+  EL_LAUNCH_CHECK("token_gate");
   return 0;
 }
 

@@ -4,7 +4,7 @@
 //             weights: the softmax over the chosen logits only.
 //   route_scored   another router on the same logits: scores s = softmax(z) over all experts, or each expert's sigmoid(z); the
 //             choice looks at s + a correction per expert, optionally only inside the `keep` groups of neighbouring experts whose
-//             best corrected score is largest; the weights are the chosen experts' s, as they are or over their sum, times a constant.  The last experts may
+//             best corrected score (or sum of the two best) is largest; the weights are the chosen experts' s, as they are or over their sum, times a constant.  The last experts may
 //             be "identity experts" without weights (they give back their input): their pairs get no row, and `combine`
 //             adds the token's own input for them.  Extra router rows after the experts give per-token gates (sigmoid).
 //   plan      the (token, choice) pairs are grouped by expert: rows of a padded layout in which every expert's rows
@@ -91,7 +91,7 @@ template <typename TH>
 __global__ void __launch_bounds__(128)
 moe_route_scored_kernel(const TH* __restrict__ h, const float* __restrict__ wr, const float* __restrict__ correction,
                         int32_t* __restrict__ idx, float* __restrict__ wts, float* __restrict__ extra, int D, int E, int n_extra, int top,
-                        int groups, int keep, float scale, int score, int renormalize) {
+                        int groups, int keep, float scale, int score, int renormalize, int group_top) {
   pdl_launch_dependents();
   pdl_wait();
   extern __shared__ float mr_smem[];         // [E + n_extra] logits, [E] choice scores, [groups] group scores, then [4][8] partial sums
@@ -124,20 +124,22 @@ moe_route_scored_kernel(const TH* __restrict__ h, const float* __restrict__ wr, 
   if (threadIdx.x >= 32) return;             // one warp chooses
   const int lane = threadIdx.x;
   if (groups > 1) {
-    if (lane == 0) {
-      const int size = E / groups;
-      for (int g = 0; g < groups; ++g) {
-        float b = -INFINITY;
-        for (int e = g * size; e < (g + 1) * size; ++e) b = fmaxf(b, c[e]);
-        gs[g] = b;
+    const int size = E / groups;
+    for (int g = lane; g < groups; g += 32) {      // a group's worth: its largest score, or the sum of its two largest
+      float b1 = -INFINITY, b2 = -INFINITY;
+      for (int e = g * size; e < (g + 1) * size; ++e) {
+        b2 = fmaxf(b2, fminf(b1, c[e]));
+        b1 = fmaxf(b1, c[e]);
       }
-      // a group is kept if fewer than `keep` groups come before it in the order (score descending, then index)
-      for (int g = 0; g < groups; ++g) {
-        int before = 0;
-        for (int o = 0; o < groups; ++o) before += (gs[o] > gs[g] || (gs[o] == gs[g] && o < g)) ? 1 : 0;
-        if (before >= keep)
-          for (int e = g * size; e < (g + 1) * size; ++e) c[e] = -INFINITY;
-      }
+      gs[g] = group_top == 2 && size > 1 ? b1 + b2 : b1;
+    }
+    __syncwarp();
+    // a group is kept if fewer than `keep` groups come before it in the order (worth descending, then index)
+    for (int g = lane; g < groups; g += 32) {
+      int before = 0;
+      for (int o = 0; o < groups; ++o) before += (gs[o] > gs[g] || (gs[o] == gs[g] && o < g)) ? 1 : 0;
+      if (before >= keep)
+        for (int e = g * size; e < (g + 1) * size; ++e) c[e] = -INFINITY;
     }
     __syncwarp();
   }
@@ -330,9 +332,61 @@ __global__ void moe_combine_kernel(float* __restrict__ x, const float* __restric
   }
 }
 
+// x[t] += rmsnorm(sum_k wts[t][k] * y[pair_row[t * top + k]] + shared[t]) * w: the weighted sum where a sublayer's output is normed
+// before the residual sum.  `shared` may be null; `xc` (may be null) receives the new x in the compute type.  A block a token; the sum
+// lies in shared memory (D floats) between its square and the scaling.
+template <typename TC>
+__global__ void moe_combine_norm_kernel(float* __restrict__ x, const float* __restrict__ y, int ldy, const float* __restrict__ wts,
+                                        const int32_t* __restrict__ pair_row, int top, int D, const float* __restrict__ shared,
+                                        const float* __restrict__ w, float eps, TC* __restrict__ xc) {
+  pdl_launch_dependents();
+  pdl_wait();
+  extern __shared__ float cn_row[];
+  __shared__ float red[33];
+  const int t = blockIdx.x;
+  float ss = 0.f;
+  for (int i = threadIdx.x; i < D; i += blockDim.x) {
+    float acc = 0.f;
+    for (int k = 0; k < top; ++k) {
+      const int r = pair_row[(size_t)t * top + k];
+      if (r >= 0) acc = fmaf(wts ? wts[(size_t)t * top + k] : 1.0f, y[(size_t)r * ldy + i], acc);
+    }
+    if (shared) acc += shared[(size_t)t * D + i];
+    cn_row[i] = acc;
+    ss = fmaf(acc, acc, ss);
+  }
+  ss = block_sum(ss, red);
+  const float inv = 1.0f / sqrtf(ss / (float)D + eps);
+  float* xr = x + (size_t)t * D;
+  for (int i = threadIdx.x; i < D; i += blockDim.x) {
+    const float nx = xr[i] + cn_row[i] * inv * w[i];
+    xr[i] = nx;
+    if (xc) xc[(size_t)t * D + i] = from_f32<TC>(nx);
+  }
+}
+
 }  // namespace edgelm
 
 using namespace edgelm;
+
+extern "C" int edgelm_moe_combine_norm(float* x, const float* y, int ldy, const float* wts, const int32_t* pair_row, int n_tokens, int top, int D,
+                                       const float* shared, const float* w, float eps, void* xc, int cast_dtype, cudaStream_t stream) {
+  if (n_tokens == 0) return 0;
+  EL_REFUSE(n_tokens > 0 && top >= 1 && D > 0 && ldy >= D && w != nullptr, "moe_combine_norm: bad sizes");
+  const size_t smem = (size_t)D * sizeof(float);
+  EL_REFUSE(smem <= 200 * 1024, "moe_combine_norm: rows of %d values", D);
+  const dim3 grid(n_tokens), block(D >= 1024 ? (n_tokens <= 64 ? 1024 : 256) : 128);
+  const int bit = pdl_bit_for_tokens(n_tokens);
+#define EL_CN(TC) do { auto kern = moe_combine_norm_kernel<TC>; \
+    if (smem > 48 * 1024) cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
+    launch_pdl(bit, kern, grid, block, smem, stream, x, y, ldy, wts, pair_row, top, D, shared, w, eps, (TC*)xc); } while (0)
+  if (xc == nullptr || cast_dtype == DT_F32) EL_CN(float);
+  else if (cast_dtype == DT_BF16) EL_CN(__nv_bfloat16);
+  else EL_REFUSE(false, "moe_combine_norm: unknown dtype code %d", cast_dtype);
+#undef EL_CN
+  EL_LAUNCH_CHECK("moe_combine_norm");
+  return 0;
+}
 
 extern "C" int edgelm_moe_tile_rows() { return MG_TM; }
 
@@ -352,17 +406,18 @@ extern "C" int edgelm_moe_route(const void* h, int dtype, const float* wr, const
 
 extern "C" int edgelm_moe_route_scored(const void* h, int dtype, const float* wr, const float* correction, int32_t* idx, float* wts,
                                        float* extra, int n_tokens, int D, int E, int n_extra, int top, int groups, int keep, float scale,
-                                       int score, int renormalize, cudaStream_t stream) {
+                                       int score, int renormalize, int group_top, cudaStream_t stream) {
   if (n_tokens == 0) return 0;
   EL_REFUSE(n_tokens > 0 && D > 0 && E >= 1 && E <= MOE_MAX_EXPERTS && top >= 1 && top <= E, "moe_route_scored: %d experts, %d chosen", E, top);
   EL_REFUSE(groups >= 1 && E % groups == 0 && keep >= 1 && keep <= groups, "moe_route_scored: %d experts in %d groups, %d kept", E, groups, keep);
+  EL_REFUSE(group_top == 1 || group_top == 2, "moe_route_scored: a group's worth from its %d largest scores", group_top);
   EL_REFUSE(n_extra >= 0 && n_extra <= 32 && (n_extra == 0 || extra != nullptr), "moe_route_scored: %d extra rows (up to 32)", n_extra);
   EL_REFUSE(score == SCORE_SOFTMAX || score == SCORE_SIGMOID, "moe_route_scored: unknown score %d", score);
   const dim3 grid(n_tokens), block(128);
   const size_t smem = (size_t)(2 * E + n_extra + groups + 32) * sizeof(float);
   const int bit = pdl_bit_for_tokens(n_tokens);
-  if (dtype == DT_F32) launch_pdl(bit, moe_route_scored_kernel<float>, grid, block, smem, stream, (const float*)h, wr, correction, idx, wts, extra, D, E, n_extra, top, groups, keep, scale, score, renormalize);
-  else if (dtype == DT_BF16) launch_pdl(bit, moe_route_scored_kernel<__nv_bfloat16>, grid, block, smem, stream, (const __nv_bfloat16*)h, wr, correction, idx, wts, extra, D, E, n_extra, top, groups, keep, scale, score, renormalize);
+  if (dtype == DT_F32) launch_pdl(bit, moe_route_scored_kernel<float>, grid, block, smem, stream, (const float*)h, wr, correction, idx, wts, extra, D, E, n_extra, top, groups, keep, scale, score, renormalize, group_top);
+  else if (dtype == DT_BF16) launch_pdl(bit, moe_route_scored_kernel<__nv_bfloat16>, grid, block, smem, stream, (const __nv_bfloat16*)h, wr, correction, idx, wts, extra, D, E, n_extra, top, groups, keep, scale, score, renormalize, group_top);
   else EL_REFUSE(false, "moe_route_scored: unknown dtype code %d", dtype);
   EL_LAUNCH_CHECK("moe_route_scored");
   return 0;

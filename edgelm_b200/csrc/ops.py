@@ -711,15 +711,53 @@ def rotate_append(qkv, bias, q_out, tok_pos, tok_seq, page_table, kcache, vcache
                                              _p(bias), _stream()))
 
 
+def norm_append(qkv, bias, q_out, tok_pos, tok_seq, page_table, kcache, vcache, nh, nkv, dk, dv, rot, interleaved, freq, err, q_norm, k_norm, eps,
+                rot_mult=1.0):
+    """`rotate_append` where a token's queries are normed over all of them (`q_norm` [nh dk]) and its keys over all of them
+    (`k_norm` [nkv dk]), `eps` inside the roots, before they are split into heads and rotated."""
+    _f32_rows(qkv, "qkv"); _f32(q_out, "q_out"); _f32(q_norm, "q_norm"); _f32(k_norm, "k_norm")
+    T = qkv.shape[0]
+    _need(qkv.shape[1] == (nh + nkv) * dk + nkv * dv and q_out.shape == (T, nh * dk), "norm_append: shapes")
+    _need(q_norm.numel() == nh * dk and k_norm.numel() == nkv * dk, "norm_append: the norms' weights")
+    _need(bias is None or (bias.dtype == torch.float32 and bias.is_contiguous() and bias.numel() == qkv.shape[1]), "norm_append: bias")
+    _need(rot == 0 or (freq is not None and freq.dtype == torch.float64 and freq.numel() == rot // 2 and freq.is_contiguous()), "norm_append: frequencies")
+    _masked_cache_check(kcache, vcache, nkv, dk, dv, "norm_append")
+    _need(vcache is not None, "norm_append: values need a cache of their own")
+    for t, n in ((tok_pos, "tok_pos"), (tok_seq, "tok_seq"), (page_table, "page_table")):
+        _i32(t, n)
+    _check(lib().edgelm_norm_append(_p(qkv), _p(bias), _p(q_out), _p(tok_pos), _p(tok_seq), _p(page_table), page_table.stride(0), kcache.shape[0],
+                                    _p(kcache), _p(vcache), _dt(kcache), T, nh, nkv, dk, dv, int(rot), 1 if interleaved else 0, _p(freq), _p(err),
+                                    _p(q_norm), _p(k_norm), ctypes.c_float(eps), qkv.stride(0), ctypes.c_float(rot_mult), _stream()))
+
+
+def latent_rows(kcache, rows, tok_pos, tok_seq, page_table, err):
+    """rows[t] = the cache row of token t of the step (one key head; rows [T, n] in the cache's type)."""
+    T, n = rows.shape
+    _need(rows.dtype == kcache.dtype and rows.is_contiguous(), "latent_rows: layout")
+    _masked_cache_check(kcache, None, 1, n, n, "latent_rows")
+    for t, nm in ((tok_pos, "tok_pos"), (tok_seq, "tok_seq"), (page_table, "page_table")):
+        _i32(t, nm)
+    _check(lib().edgelm_latent_rows(_p(kcache), _p(rows), _dt(rows), _p(tok_pos), _p(tok_seq), _p(page_table), page_table.stride(0), kcache.shape[0],
+                                    n, T, _p(err), _stream()))
+
+
 def latent_prepare(u, kv_off, has_kv, q_out, q_pitch, q_off, copy_q, norm_w, eps, tok_pos, tok_seq, page_table, kcache, nh, d, rd, r, freq, err,
-                   row_out=None, interleaved=False, rot_mult=1.0):
+                   row_out=None, interleaved=False, rot_mult=1.0, q_latent=None):
     """u [T, *] float32: nh query heads of [d | rd] from column 0 and, with `has_kv`, the latent's row [r | rd] from column
     `kv_off`.  The rotated part of every query head (pairs and `rot_mult` as in `rotate_append`) goes to q_out[t, h * q_pitch + q_off :], with
     `copy_q` the unrotated part to q_out[t, h * q_pitch :]; the latent, RMS-normed with `norm_w`, and the rotated shared key
-    part become the token's cache row [r + rd], and row t of `row_out` [T, r + rd] (optional, the cache's type)."""
-    _f32_rows(u, "u"); _f32(q_out, "q_out")
+    part become the token's cache row [r + rd], and row t of `row_out` [T, r + rd] (optional, the cache's type).  `q_latent`
+    (column, weight [n], out [T, n]): n columns of u, RMS-normed with `eps` and the weight, go to `out` in its type.  `nh` 0 (q_out
+    None): no query heads in u."""
+    _f32_rows(u, "u")
     T = u.shape[0]
-    _need(q_out.shape == (T, nh * q_pitch), "latent_prepare: q_out shape")
+    _need(nh == 0 or (q_out.dtype == torch.float32 and q_out.is_contiguous() and q_out.shape == (T, nh * q_pitch)), "latent_prepare: q_out shape")
+    kind = kcache if has_kv else None
+    if q_latent is not None:
+        ql_off, ql_w, ql_out = q_latent
+        _f32(ql_w, "q_latent weight")
+        _need(ql_out.is_contiguous() and ql_out.shape == (T, ql_w.numel()) and (kind is None or kind.dtype == ql_out.dtype), "latent_prepare: the queries' latent")
+        kind = ql_out
     _need(rd == 0 or (freq is not None and freq.dtype == torch.float64 and freq.numel() == rd // 2 and freq.is_contiguous()), "latent_prepare: frequencies")
     if has_kv:
         _f32(norm_w, "norm_w")
@@ -732,8 +770,10 @@ def latent_prepare(u, kv_off, has_kv, q_out, q_pitch, q_off, copy_q, norm_w, eps
     _check(lib().edgelm_latent_prepare(_p(u), u.stride(0), int(kv_off), 1 if has_kv else 0, _p(q_out), int(q_pitch), int(q_off), 1 if copy_q else 0,
                                        _p(norm_w) if has_kv else _p(None), ctypes.c_float(eps), _p(tok_pos), _p(tok_seq),
                                        _p(page_table) if has_kv else _p(None), page_table.stride(0) if has_kv else 0, kcache.shape[0] if has_kv else 0,
-                                       _p(kcache) if has_kv else _p(None), _p(row_out) if has_kv else _p(None), _dt(kcache) if has_kv else F32,
-                                       T, nh, d, rd, r, _p(freq), _p(err), 1 if interleaved else 0, ctypes.c_float(rot_mult), _stream()))
+                                       _p(kcache) if has_kv else _p(None), _p(row_out) if has_kv else _p(None), _dt(kind) if kind is not None else F32,
+                                       T, nh, d, rd, r, _p(freq), _p(err), 1 if interleaved else 0, ctypes.c_float(rot_mult),
+                                       int(q_latent[0]) if q_latent is not None else 0, q_latent[1].numel() if q_latent is not None else 0,
+                                       _p(q_latent[1] if q_latent is not None else None), _p(q_latent[2] if q_latent is not None else None), _stream()))
 
 
 def latent_expand_keys(kn, rows, kx, nh, d, rd, r):
@@ -762,24 +802,27 @@ def add_row_bias(x, b):
     _check(lib().edgelm_add_row_bias(_p(x), _p(b), x.shape[0], x.shape[1], _stream()))
 
 
-def _head_gate_check(gate, T, nh, what):
-    _need(gate is None or (gate.dtype == torch.float32 and gate.is_cuda and gate.shape == (T, nh) and gate.stride(1) == 1), f"{what}: the heads' gate")
+def _gate_check(gate, T, nh, dv, what):
+    """Numbers a head that an output gate has: 0 for one (gate [T, nh]), dv for one per channel (gate [T, nh dv])."""
+    _need(gate is None or (gate.dtype == torch.float32 and gate.is_cuda and gate.shape in ((T, nh), (T, nh * dv)) and gate.stride(1) == 1), f"{what}: the heads' gate")
+    return dv if gate is not None and dv > 1 and gate.shape[1] == nh * dv else 0
 
 
 def masked_attn(q, out, kcache, vcache, tok_pos, tok_seq, page_table, nh, nkv, dk, dv, scale, mask, mask_size, sink, max_keys, maps=1, gate=None,
-                n_splits=1, part=None):
+                n_splits=1, part=None, keep=0):
     """Attention of every token of the step over the keys lo .. its position (`mask`: MASK_CAUSAL lo = 0; MASK_WINDOW the
     last `mask_size` keys; MASK_CHUNK the keys of its own chunk of `mask_size` positions).  q [T, nh dk] float32; out
     [T, nh dv] float32 or the cache's type; `vcache` None: a value is the first dv dimensions of its key row.  `sink`
     (float32 [nh] or None): one more term exp(sink_h) in the denominator.  `max_keys`: the most keys a token sees.
     `maps` > 1: every query head and key row holds `maps` runs of dk dimensions, each an attention of its own over the
     head's values: q [T, nh maps dk], key rows of maps dk, out [T, nh maps dv] (no sink then).  `gate` (float32 [T, nh], rows of
-    any pitch): head h's output is multiplied by sigmoid(gate[t, h]) before it is rounded.  `n_splits` > 1: a token's keys are
+    any pitch): head h's output is multiplied by sigmoid(gate[t, h]) before it is rounded; [T, nh dv]: every channel by its own.
+    `keep` (with MASK_WINDOW): the sequence's first `keep` keys stay visible behind the window.  `n_splits` > 1: a token's keys are
     dealt to so many blocks, whose partial results go through `part` (float32, T nh maps n_splits (2 + dv) values) and are
     merged by a second launch: for steps of few tokens over long sequences."""
     _f32(q, "q")
     T = q.shape[0]
-    _head_gate_check(gate, T, nh, "masked_attn")
+    gate_ch = _gate_check(gate, T, nh, dv, "masked_attn")
     _need(n_splits == 1 or (part is not None and part.dtype == torch.float32 and part.is_contiguous() and part.numel() >= T * nh * maps * n_splits * (2 + dv)),
           "masked_attn: room for the splits' partial results")
     _need(q.shape == (T, nh * maps * dk) and out.is_contiguous() and out.shape == (T, nh * maps * dv), "masked_attn: shapes")
@@ -790,8 +833,8 @@ def masked_attn(q, out, kcache, vcache, tok_pos, tok_seq, page_table, nh, nkv, d
         _i32(t, n)
     _check(lib().edgelm_masked_attn(_p(q), _p(out), _dt(out), _p(kcache), _p(vcache), _dt(kcache), _p(tok_pos), _p(tok_seq), _p(page_table),
                                     page_table.stride(0), kcache.shape[0], T, nh, nkv, dk, dv, ctypes.c_float(scale), int(mask), int(mask_size or 0),
-                                    _p(sink), int(max_keys), int(maps), _p(gate), gate.stride(0) if gate is not None else 0, int(n_splits), _p(part), _stream()),
-           launches=2 if n_splits > 1 else 1)
+                                    _p(sink), int(max_keys), int(maps), _p(gate), gate.stride(0) if gate is not None else 0, int(n_splits), _p(part),
+                                    int(keep), gate_ch, _stream()), launches=2 if n_splits > 1 else 1)
 
 
 def masked_attn_tiled_takes(dk, dv, own_values=True):
@@ -801,16 +844,16 @@ def masked_attn_tiled_takes(dk, dv, own_values=True):
 
 
 def masked_attn_tiled(q, out, kcache, vcache, page_table, tile_seq, tile_tok0, tile_ntok, tile_pos0, n_tiles, max_tile_tokens, nh, nkv,
-                      dk, dv, scale, mask, mask_size, sink, n_splits=1, part=None, maps=1, gate=None):
+                      dk, dv, scale, mask, mask_size, sink, n_splits=1, part=None, maps=1, gate=None, keep=0):
     """`masked_attn` for prompt steps: the step's tokens come as tiles (runs of at most `max_tile_tokens` consecutive tokens of
     one sequence); a page of keys and values is staged once for all the rows of a tile.  `page_table` None: `kcache` [T, nkv dk]
     and `vcache` [T, nkv dv] are the step's own keys and values, and every sequence of the step starts at position 0.
     `n_splits` > 1: the pages that a tile sees are dealt to so many blocks, whose partial results go through `part` (float32,
     T nh n_splits (2 + dv) values) and are merged by a second launch: for steps of few tokens over long sequences.
-    `maps` and `gate` as in `masked_attn` (then `part` holds T nh maps n_splits (2 + dv) values)."""
+    `maps`, `gate` and `keep` as in `masked_attn` (then `part` holds T nh maps n_splits (2 + dv) values)."""
     _f32(q, "q")
     T = q.shape[0]
-    _head_gate_check(gate, T, nh, "masked_attn_tiled")
+    gate_ch = _gate_check(gate, T, nh, dv, "masked_attn_tiled")
     _need(q.shape == (T, nh * maps * dk) and out.is_contiguous() and out.shape == (T, nh * maps * dv), "masked_attn_tiled: shapes")
     _need(maps == 1 or (sink is None and vcache is not None), "masked_attn_tiled: several maps take no sink and values of their own")
     if page_table is not None:
@@ -828,7 +871,7 @@ def masked_attn_tiled(q, out, kcache, vcache, page_table, tile_seq, tile_tok0, t
                                           page_table.stride(0) if page_table is not None else 0, kcache.shape[0] if page_table is not None else 0,
                                           _p(tile_seq), _p(tile_tok0), _p(tile_ntok), _p(tile_pos0), int(n_tiles),
                                           int(max_tile_tokens), nh, nkv, dk, dv, ctypes.c_float(scale), int(mask), int(mask_size or 0), _p(sink),
-                                          int(n_splits), _p(part), T, int(maps), _p(gate), gate.stride(0) if gate is not None else 0, _stream()),
+                                          int(n_splits), _p(part), T, int(maps), _p(gate), gate.stride(0) if gate is not None else 0, int(keep), gate_ch, _stream()),
            launches=2 if n_splits > 1 else 1)
 
 
@@ -841,10 +884,10 @@ def attn_prefill_split_takes(dtype, dk, dv):
 
 
 def attn_prefill_split(q, out, kcache, vcache, page_table, tile_seq, tile_tok0, tile_ntok, tile_pos0, n_tiles, nh, nkv, dk, dv, scale, gate=None,
-                       max_keys=0, mask=0, mask_size=0, sink=None):
+                       max_keys=0, mask=0, mask_size=0, sink=None, keep=0):
     """Attention of a prompt step over bfloat16 keys and values on the tensor cores with float32 scores and softmax weights: the
     float32 operand of each product (queries; weights) goes as three bfloat16 terms.  q [T, nh dk] float32; out [T, nh dv]
-    bfloat16; tiles of at most SPLIT_PREFILL_TILE tokens; `page_table`, `mask`, `mask_size`, `sink` and `gate` as in
+    bfloat16; tiles of at most SPLIT_PREFILL_TILE tokens; `page_table`, `mask`, `mask_size`, `sink`, `gate` and `keep` as in
     `masked_attn_tiled` (`page_table` None: the step's own rows, every sequence from position 0)."""
     _f32(q, "q")
     T = q.shape[0]
@@ -856,13 +899,13 @@ def attn_prefill_split(q, out, kcache, vcache, page_table, tile_seq, tile_tok0, 
     else:
         _need(kcache.is_contiguous() and vcache.is_contiguous() and kcache.shape == (T, nkv * dk) and vcache.shape == (T, nkv * dv), "attn_prefill_split: the step's own keys and values")
     _need(sink is None or (sink.dtype == torch.float32 and sink.is_cuda and sink.is_contiguous() and sink.numel() == nh), "attn_prefill_split: sink")
-    _head_gate_check(gate, T, nh, "attn_prefill_split")
+    gate_ch = _gate_check(gate, T, nh, dv, "attn_prefill_split")
     for t, n in ((tile_seq, "tile_seq"), (tile_tok0, "tile_tok0"), (tile_ntok, "tile_ntok"), (tile_pos0, "tile_pos0")):
         _i32(t, n)
     _check(lib().edgelm_attn_prefill_split(_p(q), q.stride(0), _p(out), out.stride(0), _p(kcache), _p(vcache), _p(page_table),
                                            page_table.stride(0) if page_table is not None else 0, _p(tile_seq), _p(tile_tok0), _p(tile_ntok), _p(tile_pos0),
                                            int(n_tiles), nh, nkv, dk, dv, ctypes.c_float(scale), int(mask), int(mask_size or 0), _p(sink),
-                                           _p(gate), gate.stride(0) if gate is not None else 0, int(max_keys), _stream()))
+                                           _p(gate), gate.stride(0) if gate is not None else 0, int(max_keys), int(keep), gate_ch, _stream()))
 
 
 # ----------------------------------------------------------------------------- gated delta rule
@@ -912,13 +955,15 @@ def moe_route(h, wr, br, idx, wts, top):
 
 
 ROUTER_SCORES = {"softmax": 0, "sigmoid": 1}
+GROUP_SCORES = {"max": 1, "top2_sum": 2}
 
 
-def moe_route_scored(h, wr, correction, idx, wts, top, n_experts, groups=1, keep=1, scale=1.0, extra=None, score="softmax", renormalize=True):
+def moe_route_scored(h, wr, correction, idx, wts, top, n_experts, groups=1, keep=1, scale=1.0, extra=None, score="softmax", renormalize=True,
+                     group_score="max"):
     """The router that scores every expert: s = softmax(wr[:n_experts] h) over all experts, or sigmoid(wr[e] h) expert by expert
     (float32); the `top` experts with the
     largest s + correction are chosen (first of equal ones), with `groups` > 1 only among the `keep` groups of neighbouring
-    experts whose best corrected score is largest (the others count as minus infinity: when the kept groups hold fewer than `top`
+    experts whose best corrected score (`group_score` "max") or sum of the two best ("top2_sum") is largest (the others count as minus infinity: when the kept groups hold fewer than `top`
     experts, the left-out ones follow in the order of their numbers); wts = s of the chosen over their sum (+ 1e-20; not
     `renormalize`: s as it is), times `scale`.  Rows of `wr` after the first `n_experts` give `extra` [T, rows] = sigmoid(row . h).  idx of a choice that could not
     be made (scores that are not numbers): -1."""
@@ -929,7 +974,8 @@ def moe_route_scored(h, wr, correction, idx, wts, top, n_experts, groups=1, keep
     _need(correction is None or (correction.dtype == torch.float32 and correction.is_contiguous() and correction.numel() == n_experts), "moe_route_scored: correction")
     _need((n_extra == 0) == (extra is None) and (extra is None or (extra.dtype == torch.float32 and extra.is_contiguous() and extra.shape == (T, n_extra))), "moe_route_scored: extra rows")
     _check(lib().edgelm_moe_route_scored(_p(h), _dt(h), _p(wr), _p(correction), _p(idx), _p(wts), _p(extra), T, D, int(n_experts), int(n_extra), int(top),
-                                         int(groups), int(keep), ctypes.c_float(scale), ROUTER_SCORES[score], 1 if renormalize else 0, _stream()))
+                                         int(groups), int(keep), ctypes.c_float(scale), ROUTER_SCORES[score], 1 if renormalize else 0, GROUP_SCORES[group_score],
+                                         _stream()))
 
 
 def moe_plan(idx, n_experts, tile_rows, row_pair, pair_row, tile_expert):
@@ -1024,6 +1070,23 @@ def moe_combine(x, y, wts, pair_row, idx=None, n_real=0, h=None, shared=None, ga
         _need(shared.shape == (T, D) and (gate is None or (gate.dtype == torch.float32 and gate.is_contiguous() and gate.numel() == T)), "moe_combine: the shared term")
     _check(lib().edgelm_moe_combine(_p(x), _p(y), y.stride(0), _p(wts), _p(pair_row), T, top, D, _p(idx), int(n_real), _p(h if idx is not None else None),
                                     _dt(h) if idx is not None else F32, _p(shared), _p(gate if shared is not None else None), _stream()))
+
+
+def moe_combine_norm(x, y, wts, pair_row, w, eps, shared=None, cast=None, top=None):
+    """x += rmsnorm(sum_k wts[t, k] * y[pair_row[t * top + k]] + shared[t]) * w in one pass (`wts` None with `top` given: every weight
+    is 1); `cast` (optional, [T, D] in the compute dtype) receives the new x too."""
+    _f32(x, "x"); _f32(y, "y"); _f32(w, "w"); _i32(pair_row, "pair_row")
+    T, D = x.shape
+    if wts is not None:
+        _f32(wts, "wts")
+        top = wts.shape[1]
+    _need(top is not None and (wts is None or wts.shape[0] == T) and y.shape[1] == D and pair_row.numel() == T * top and w.numel() == D, "moe_combine_norm: shapes")
+    if shared is not None:
+        _f32(shared, "shared")
+        _need(shared.shape == (T, D), "moe_combine_norm: the shared term")
+    _need(cast is None or (cast.shape == x.shape and cast.is_contiguous()), "moe_combine_norm: the copy's layout")
+    _check(lib().edgelm_moe_combine_norm(_p(x), _p(y), y.stride(0), _p(wts), _p(pair_row), T, int(top), D, _p(shared), _p(w), ctypes.c_float(eps),
+                                         _p(cast), _dt(cast) if cast is not None else F32, _stream()))
 
 
 # ----------------------------------------------------------------------------- several residual streams
@@ -1200,6 +1263,15 @@ def rmsnorm_pair(x, w1, eps, y1, w2=None, y2=None, add=None):
                                                             y2.shape == x.shape and y2.is_contiguous() and y2.dtype == y1.dtype)), "rmsnorm_pair: the second norm")
     _need(add is None or (add.dtype == torch.float32 and add.is_contiguous() and add.shape == x.shape), "rmsnorm_pair: the rows to add")
     _check(lib().edgelm_rmsnorm_pair(_p(x), _p(add), _p(w1), _p(w2), _p(y1), _p(y2), _dt(y1), x.shape[0], x.shape[1], ctypes.c_float(eps), _stream()))
+
+
+def token_gate(u, ids, table, out, err):
+    """out[t] = gelu_tanh(u[t]) * table[ids[t]] (u [T, n] float32, table [vocab, n] and out [T, n] in the compute dtype); ids outside
+    the table set bit 1 of `err`."""
+    _f32(u, "u"); _i32(ids, "ids")
+    T, n = u.shape
+    _need(out.shape == (T, n) and out.is_contiguous() and table.is_contiguous() and table.dtype == out.dtype and table.shape[1] == n and ids.numel() == T, "token_gate: shapes")
+    _check(lib().edgelm_token_gate(_p(u), _p(ids), _p(table), _p(out), _dt(out), T, n, table.shape[0], _p(err), _stream()))
 
 
 def softcap(z, cap):

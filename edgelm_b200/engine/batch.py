@@ -60,6 +60,9 @@ class StepContext:
         # models that carry several residual streams: the read that the running layer's last write should also do
         # ((in-weights, norm weight, eps, output, whether it is the next layer's input) or None), and the next layer's input if done
         self.streams_next = self.streams_h = None
+        # models with layers that read the residual stream itself: the buffer for x in the compute dtype that such layers share (or
+        # None), whether it holds the x that the next layer starts from, and whether the next layer would read it
+        self.x_cast, self.x_cast_ready, self.x_cast_wanted = None, False, False
         self.rows_to_add = None        # rows that the next layer adds to the residual stream before anything else (or None)
         self.token_ids = self.tok_pos = self.tok_seq = self.seq_index = self.seq_pos = self.want_rows = None
         self.seq_tok0 = None           # packed row of each sequence's first token, then the token count (int32 [n_seqs + 1])

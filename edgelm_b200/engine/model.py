@@ -34,6 +34,8 @@ class DecoderModel:
         self.carry = any(hasattr(l, "first_read") for l in self.layers)
         if self.carry != all(hasattr(l, "first_read") for l in self.layers) or (self.streams > 1 and not self.carry):
             raise ConfigError(f"a plan with {self.streams} residual streams needs layer arrangements that all carry them")
+        # layers that read the residual stream itself share a copy of it in the compute dtype, which each leaves to the next
+        self.shares_cast = dtype != torch.float32 and any(getattr(l, "takes_cast", False) for l in self.layers)
         self.keeps_embedding = any(e.add_embedding for e in self.schedule)      # a copy of the embedding's output outlives the layers
         for i, e in enumerate(self.schedule):
             need = self.layers[e.layer].cache_need()
@@ -94,6 +96,8 @@ class DecoderModel:
         x = nbytes((n_tokens, d), torch.float32) * (2 if self.keeps_embedding else 1)
         if self.carry:
             x += nbytes((n_tokens, self.streams, d), torch.float32) + nbytes((n_tokens, d), self.dtype)
+        if self.shares_cast:
+            x += nbytes((n_tokens, d), self.dtype)
         layers = max(l.workspace_bytes(n_tokens, n_seqs) for l in self.layers)
         head = nbytes((n_want, d), self.dtype)
         return x + max(layers, head) + 4096
@@ -168,12 +172,15 @@ class DecoderModel:
             with ctx.prof("streams"):
                 ops.streams_fill(x, carried)
             ctx.streams_h = None
+        ctx.x_cast = ws.alloc((T, self.plan.hidden_size), self.dtype) if self.shares_cast else None
+        ctx.x_cast_ready = False
         for i, e in enumerate(self.schedule):
             entry = cache.entries[e.reads_cache_of if e.reads_cache_of is not None else i]
             nxt = self.schedule[i + 1].layer if i + 1 < len(self.schedule) else None
             ctx.weights_after = self.layers[nxt].first_weights() if nxt is not None else ()
             if self.carry:
                 ctx.streams_next = (*self.layers[nxt].first_read(), h_next, True) if nxt is not None else (self._ones, None, 0.0, x, False)
+            ctx.x_cast_wanted = nxt is not None and getattr(self.layers[nxt], "takes_cast", False) and not self.schedule[i + 1].add_embedding
             # (the embedding's output joining the stream again: the layer's first pass over x does it, if its arrangement
             # can (`takes_added_rows`), else a pass of its own)
             ctx.rows_to_add = x0 if e.add_embedding else None

@@ -1,6 +1,6 @@
 """Arrangements of one layer's parts.  "prenorm": x += mixer(norm1(x)); x += ffn(norm2(x))
 (adarsh-sgh/edgelm tools/elm.py:122-153); a layer may have no feed-forward.  "sublayer_norm": x += norm1(mixer(x)); x += norm2(ffn(x)), with an
-optional blend of the mixer's input with the previous token's.  "parallel_prenorm": x += mixer(norm1(x)) + ffn(norm2(x)), both
+optional blend of the mixer's input with the previous token's and further sublayers of the same form.  "parallel_prenorm": x += mixer(norm1(x)) + ffn(norm2(x)), both
 sublayers reading the same x.  "hyper": the pre-norm arrangement over several copies of the
 residual stream, which every sublayer reads through learned weights and rewrites through a learned matrix."""
 import torch
@@ -143,8 +143,10 @@ class SublayerNormBlock(Part):
     residual stream itself.  With the option `shift` (a tensor's name) the mixer's input is first blended with the
     previous token's: h_t = x_t + (x_(t-1) - x_t) * shift, element by element, with zeros before a sequence's first
     token; the last x of every sequence is then part of its state (a float32 row of its own beside the mixer's).
-    A layer may have no feed-forward.  Mixers and feed-forwards are asked to STORE their output (`accumulate=False`):
-    the residual sum is the norm kernel's, which also hands the feed-forward its input in the compute dtype."""
+    A layer may have no feed-forward.  The option `after` lists more sublayers, (feed-forward, norm) specs, that follow the
+    feed-forward in the same form.  Mixers and feed-forwards are asked to STORE their output (`accumulate=False`):
+    the residual sum is the norm kernel's (or the feed-forward's own last kernel's, if it takes the norm), which also hands the
+    next sublayer its input in the compute dtype, the next layer's too (`ctx.x_cast`)."""
 
     def __init__(self, layer_spec, env):
         self.prefix = layer_spec.prefix
@@ -153,13 +155,21 @@ class SublayerNormBlock(Part):
         self.mixer = env.build("mixer", layer_spec.mixer)
         self.ffn = env.build("ffn", layer_spec.ffn) if layer_spec.ffn is not None else None
         self.ffn_norm = env.build("norm", layer_spec.ffn_norm) if layer_spec.ffn is not None else None
-        for n in (self.mixer_norm, self.ffn_norm):
-            if n is not None and not hasattr(n, "add_normed"):
+        self.ffns = [] if self.ffn is None else [(self.ffn, self.ffn_norm)]
+        self.ffns += [(env.build("ffn", f), env.build("norm", n)) for f, n in layer_spec.options.get("after") or ()]
+        for n in [self.mixer_norm] + [n for _, n in self.ffns]:
+            if not hasattr(n, "add_normed"):
                 raise ConfigError(f"block 'sublayer_norm': the norm '{n.kind}' cannot be applied to a sublayer's output (no add_normed)")
-        self.parts = tuple(p for p in (self.mixer_norm, self.mixer, self.ffn_norm, self.ffn) if p is not None)
+        self.parts = (self.mixer_norm, self.mixer) + tuple(p for f, n in self.ffns for p in (n, f))
         self.hidden = layer_spec.mixer_norm["dim"]
         self.shift_name = layer_spec.options.get("shift")
+        self.unused_norm = layer_spec.options.get("unused_norm") if self.ffn is None else None
         self.shift = None
+        self.takes_cast = self.shift_name is None      # the mixer reads x itself: the layer before may leave it in the compute dtype
+
+    def ignorable(self):
+        """A layer without a feed-forward may still come with its norm's weight in the files."""
+        return (self.prefix + self.unused_norm,) if self.unused_norm else ()
 
     def weight_shapes(self, prefix=None):
         out = {}
@@ -180,9 +190,8 @@ class SublayerNormBlock(Part):
 
     def sizes(self):
         out = {}
-        for p in (self.mixer, self.ffn, self.mixer_norm):
-            if p is not None:
-                out.update(p.sizes())
+        for p in [self.mixer] + [f for f, _ in self.ffns] + [self.mixer_norm]:
+            out.update(p.sizes())
         out["token_shift"] = bool(self.shift_name)
         return out
 
@@ -190,7 +199,7 @@ class SublayerNormBlock(Part):
         return sum(p.flops(n_tokens, attended) for p in self.parts)
 
     def describe(self):
-        ffn = f"; x += {self.ffn_norm.describe()}({self.ffn.describe()})" if self.ffn is not None else ""
+        ffn = "".join(f"; x += {n.describe()}({f.describe()})" for f, n in self.ffns)
         return f"{self.kind}{' with token shift' if self.shift_name else ''}: x += {self.mixer_norm.describe()}({self.mixer.describe()}){ffn}"
 
     def tile_sizes(self):
@@ -201,8 +210,8 @@ class SublayerNormBlock(Part):
         return all(p.graph_safe for p in self.parts)
 
     def workspace_bytes(self, n_tokens, n_seqs):
-        inner = max(self.mixer.workspace_bytes(n_tokens, n_seqs), self.ffn.workspace_bytes(n_tokens, n_seqs) if self.ffn is not None else 0)
-        return nbytes((n_tokens, self.hidden), self.dtype) + nbytes((n_tokens, self.hidden), torch.float32) + inner
+        inner = max(p.workspace_bytes(n_tokens, n_seqs) for p in [self.mixer] + [f for f, _ in self.ffns])
+        return 2 * nbytes((n_tokens, self.hidden), self.dtype) + nbytes((n_tokens, self.hidden), torch.float32) + inner
 
     def first_weights(self):
         return self.mixer.first_weights()
@@ -210,31 +219,40 @@ class SublayerNormBlock(Part):
     def forward(self, ctx, x, cache):
         T, ws = x.shape[0], ctx.ws
         after_layer = ctx.weights_after
+        full = self.dtype == torch.float32
         with ws.frame():
-            h = ws.alloc((T, self.hidden), self.dtype)      # the mixer's input; later the feed-forward's
+            # x in the compute dtype, what every sublayer reads: the model's buffer for the layers that hand it on, or one of this layer's
+            h = x if full else (ctx.x_cast if ctx.x_cast is not None else ws.alloc((T, self.hidden), self.dtype))
             y = ws.alloc((T, self.hidden), torch.float32)   # a sublayer's output before its norm
             if self.shift is not None:
-                state = cache["shift"].state
+                state, mixer_in = cache["shift"].state, ws.alloc((T, self.hidden), self.dtype)
                 with ctx.prof("token_shift"):
-                    ops.shift_mix(x, state, self.shift, h.view(1, T, self.hidden), ctx.tok_seq, ctx.seq_tok0, ctx.seq_slots, move_state=True)
-                mixer_in = h
-            elif self.dtype == torch.float32:
-                mixer_in = x
+                    ops.shift_mix(x, state, self.shift, mixer_in.view(1, T, self.hidden), ctx.tok_seq, ctx.seq_tok0, ctx.seq_slots, move_state=True)
             else:
-                h.copy_(x)
                 mixer_in = h
-            ctx.weights_after = self.ffn.first_weights() if self.ffn is not None else after_layer
+                if not full and not ctx.x_cast_ready:
+                    h.copy_(x)
+            ctx.x_cast_ready = False
+            ctx.weights_after = self.ffns[0][0].first_weights() if self.ffns else after_layer
             with ws.frame():
                 self.mixer.forward(ctx, mixer_in, y, cache.get("mixer"), accumulate=False)
-            ctx.weights_after = after_layer
-            feeds = self.ffn is not None and self.dtype != torch.float32
+            hand_on = ctx.x_cast_wanted and ctx.x_cast is not None
+            cast = h if not full and (self.ffns or hand_on) else None
             with ctx.prof("norm_residual"):
-                self.mixer_norm.add_normed(ctx, x, y, cast=h if feeds else None)
-            if self.ffn is not None:
+                self.mixer_norm.add_normed(ctx, x, y, cast=cast)
+            for i, (ffn, norm) in enumerate(self.ffns):
+                last = i + 1 == len(self.ffns)
+                ctx.weights_after = after_layer if last else self.ffns[i + 1][0].first_weights()
+                cast = h if not full and (not last or hand_on) else None
                 with ws.frame():
-                    self.ffn.forward(ctx, h if feeds else x, y, accumulate=False)
+                    if hasattr(ffn, "takes_norm") and ffn.takes_norm(norm):
+                        ffn.forward(ctx, h, x, norm=norm, cast=cast)
+                        continue
+                    ffn.forward(ctx, h, y, accumulate=False)
                 with ctx.prof("norm_residual"):
-                    self.ffn_norm.add_normed(ctx, x, y)
+                    norm.add_normed(ctx, x, y, cast=cast)
+            ctx.x_cast_ready = hand_on and not full
+            ctx.weights_after = after_layer
 
 
 @register_block("hyper")

@@ -8,6 +8,7 @@ stretched (`parts.rope.rotary_frequencies`, `rotary_magnitude`).  score = (q . k
 
     causal   position i sees every j <= i
     window   the last `size` keys, its own included
+             (with `keep_first` k the sequence's first k keys stay visible behind the window, at their own positions)
     chunk    the j <= i of its own chunk, floor(i / size) = floor(j / size), counted from the sequence's first position
 
 With `sink` (a tensor's name) the softmax's denominator has one more term exp(sink_h) per query head, which has no key
@@ -19,7 +20,8 @@ Options, each with its constants in the spec:
               out_t[c] = sum_j taps[c, j] * in_(t - conv + 1 + j)[c], no bias, inputs from before a sequence's start
               counting as zero; the filter's memory, the previous conv - 1 projected rows, is kept per sequence as state
     qk_norm   {eps}: every query and key head (every map of it) is divided by its root mean square and multiplied by a
-              weight of head_dim values that all heads share (`q_norm`, `k_norm`), before the rotation
+              weight of head_dim values that all heads share (`q_norm`, `k_norm`), before the rotation; {eps, "over": "projection"}:
+              all of a token's queries are divided by their common root mean square, all its keys by theirs, with a weight per row
     diff      {offset, eps}: "differential" attention.  A head has two maps, each with queries and keys of head_dim of its
               own (q and k rows laid out head by head as [map 1, map 2]) and a softmax of its own over the same values.
               With lambda = exp(lq1 . lk1) - exp(lq2 . lk2) + offset (four tensors of head_dim, one number per layer):
@@ -27,6 +29,7 @@ Options, each with its constants in the spec:
     head_gate True: one more projection of the mixer's input with one row per query head (`names["gate"]`, no bias); head h's
               output is multiplied by the sigmoid of its number before the output projection.  The rows ride in the stacked
               q, k, v product; the attention kernels multiply before they round.
+    channel_gate  True: the same with a row per channel of the heads' outputs: every channel is multiplied by its own sigmoid
 """
 import torch
 
@@ -53,10 +56,18 @@ def read_mask(mask, where):
     return MASKS[kind], size
 
 
-def most_keys(mask, size):
+def kept_first(mask, where):
+    """How many of a sequence's first keys stay visible behind a window (0: none)."""
+    keep = int((mask or {}).get("keep_first") or 0)
+    if keep < 0 or (keep and mask.get("kind") != "window"):
+        raise ConfigError(f"{where}: {keep} kept first keys behind a mask of kind '{mask.get('kind', 'causal')}'")
+    return keep
+
+
+def most_keys(mask, size, keep=0):
     """The most keys that a token can see under the mask (a bound that does not depend on the step: the choice it
     drives is frozen into a captured graph)."""
-    return size if mask != ops.MASK_CAUSAL else 1 << 30
+    return size + keep if mask != ops.MASK_CAUSAL else 1 << 30
 
 
 # Steps of one token a sequence: with at least so many query heads to a key head the tiled kernel is used (a tile = one
@@ -75,9 +86,9 @@ BLOCKS_AN_SM = 4        # (8 sequences of 32 heads over 2,048 keys, a decode ste
 SHARED_KEYS_LONG_GROUP = 3
 
 
-def head_splits(ctx, n_pairs, mask, mask_size):
+def head_splits(ctx, n_pairs, mask, mask_size, keep=0):
     """Blocks that share a (token, head) pair's keys in the block-per-pair kernel: about BLOCKS_AN_SM blocks of four warps an SM."""
-    if most_keys(mask, mask_size) <= SPLIT_KEYS_FROM:
+    if most_keys(mask, mask_size, keep) <= SPLIT_KEYS_FROM:
         return 1
     return min(MAX_HEAD_SPLITS, max(1, (BLOCKS_AN_SM * ctx.n_sms + n_pairs - 1) // max(1, n_pairs)))
 MAX_SPLITS = 32
@@ -93,12 +104,12 @@ def single_token_tiles(ctx):
     return ctx.seq_index, ctx.seq_index, _ones[key][:ctx.n_seqs], ctx.tok_pos
 
 
-def decode_splits(ctx, n_kv_heads, group, mask, mask_size):
+def decode_splits(ctx, n_kv_heads, group, mask, mask_size, keep=0):
     """Blocks that share a token's pages in the tiled kernel: about two blocks an SM, at most a block a page of the mask."""
     tiles = max(1, ctx.n_seqs * n_kv_heads * ((group + 31) // 32))
     splits = min(MAX_SPLITS, max(1, (2 * ctx.n_sms + tiles - 1) // tiles))
     if mask != ops.MASK_CAUSAL:
-        splits = min(splits, (mask_size + 63) // 64 + 1)
+        splits = min(splits, (mask_size + 63) // 64 + 1 + (keep + 63) // 64)
     return splits
 
 
@@ -126,6 +137,7 @@ class MaskedAttention(Part):
         self.taps = int(spec.get("conv") or 0)                    # 0: no convolution
         self.qk_norm, self.diff = spec.get("qk_norm"), spec.get("diff")
         self.head_gate = bool(spec.get("head_gate", False))
+        self.channel_gate = bool(spec.get("channel_gate", False))
         self.maps = 2 if self.diff else 1
         self.names = dict(spec["names"])
         self.dtype = env.dtype
@@ -135,14 +147,21 @@ class MaskedAttention(Part):
             raise ConfigError(f"masked_attention: head sizes {self.dk} / {self.dv} are not taken (key rows to 1024, values to 512)")
         if self.diff and "sink" in self.names:
             raise ConfigError("masked_attention: differential maps take no sink")
-        if self.diff and self.head_gate:
-            raise ConfigError("masked_attention: differential maps take no gate per head")
+        if self.diff and (self.head_gate or self.channel_gate):
+            raise ConfigError("masked_attention: differential maps take no gate per head or channel")
+        if self.head_gate and self.channel_gate:
+            raise ConfigError("masked_attention: a gate per head and one per channel at once are not taken")
+        self.norm_all = bool(self.qk_norm) and self.qk_norm.get("over", "head") == "projection"
+        if self.norm_all and (self.diff or self.taps or (self.nh + self.nkv) * self.dk > 50 * 1024):
+            raise ConfigError("masked_attention: a norm over the whole projection goes with one map a head, no filter, and rows to 51,200 values")
         if self.rot % 2 or not 0 <= self.rot <= self.dk:
             raise ConfigError(f"masked_attention: {self.rot} rotated dimensions of a head of {self.dk}")
         self.mask, self.mask_size = read_mask(spec.get("mask"), "masked_attention")
+        self.keep = kept_first(spec.get("mask"), "masked_attention")
         self.kw = self.dk * self.maps                                # what a head's queries and a key row hold
         self.d_qkv = (self.nh + self.nkv) * self.kw + self.nkv * self.dv
-        self.d_in = self.d_qkv + (self.nh if self.head_gate else 0)     # columns of the stacked product: q | k | v | gate
+        self.d_gate = self.nh if self.head_gate else (self.nh * self.dv if self.channel_gate else 0)
+        self.d_in = self.d_qkv + self.d_gate     # columns of the stacked product: q | k | v | gate
         self.tile_tokens = max(1, 32 // (self.nh // self.nkv))
         self.freq = self.b_qkv = self.b_o = self.sink = self.conv_w = self.q_norm = self.k_norm = self.no_tail = None
         self.lam = 0.0
@@ -182,15 +201,19 @@ class MaskedAttention(Part):
         if self.diff:
             out["diff_offset"] = float(self.diff["offset"])
         if self.qk_norm:
-            out["qk_norm"] = True
+            out["qk_norm"] = "projection" if self.norm_all else True
         if self.head_gate:
             out["head_gate"] = True
+        if self.channel_gate:
+            out["channel_gate"] = True
+        if self.keep:
+            out["kept_first"] = self.keep
         return out
 
     def flops(self, n_tokens, attended):
         proj = 2.0 * n_tokens * self.hidden * (self.d_in + self.nh * self.dv)
         if self.mask != ops.MASK_CAUSAL:
-            attended = min(attended, n_tokens * self.mask_size)
+            attended = min(attended, n_tokens * (self.mask_size + self.keep))
         return proj + 2.0 * attended * self.nh * self.maps * (self.dk + self.dv)
 
     def weight_shapes(self, prefix):
@@ -198,8 +221,8 @@ class MaskedAttention(Part):
         rows = {"q": self.nh * self.kw, "k": self.nkv * self.kw, "v": self.nkv * self.dv}
         out = {prefix + n[k]: (r, self.hidden) for k, r in rows.items()}
         out[prefix + n["o"]] = (self.hidden, self.nh * self.dv)
-        if self.head_gate:
-            out[prefix + n["gate"]] = (self.nh, self.hidden)
+        if self.d_gate:
+            out[prefix + n["gate"]] = (self.d_gate, self.hidden)
         if self.bias:
             out.update({prefix + n[k] + n["bias"]: (r,) for k, r in rows.items()})
         if self.out_bias:
@@ -209,14 +232,15 @@ class MaskedAttention(Part):
         if self.taps:
             out.update({prefix + n[k] + n["conv"]: (r, self.taps) for k, r in rows.items()})
         if self.qk_norm:
-            out.update({prefix + n["q_norm"]: (self.dk,), prefix + n["k_norm"]: (self.dk,)})
+            out.update({prefix + n["q_norm"]: (self.nh * self.dk if self.norm_all else self.dk,),
+                        prefix + n["k_norm"]: (self.nkv * self.dk if self.norm_all else self.dk,)})
         if self.diff:
             out.update({prefix + n[k]: (self.dk,) for k in ("lq1", "lk1", "lq2", "lk2")})
         return out
 
     def load(self, tensors, prefix, device):
         n = self.names
-        stacked = ("q", "k", "v", "gate") if self.head_gate else ("q", "k", "v")
+        stacked = ("q", "k", "v", "gate") if self.d_gate else ("q", "k", "v")
         self.w_qkv = torch.cat([as_matrix(tensors[prefix + n[k]], self.dtype, device) for k in stacked], dim=0).contiguous()
         self.w_o = as_matrix(tensors[prefix + n["o"]], self.dtype, device)
         if self.bias:
@@ -266,7 +290,7 @@ class MaskedAttention(Part):
             with ctx.prof("qkv_proj"):
                 linear.matmul(ctx, h, self.w_qkv, u, prefetch=(self.w_o,))
         qkv = u[:, :self.d_qkv]
-        gate = u[:, self.d_qkv:] if self.head_gate else None
+        gate = u[:, self.d_qkv:] if self.d_gate else None
         bias = self.b_qkv
         conv = None
         if self.taps:       # (the filter over time runs inside the kernel that norms, rotates and appends)
@@ -275,38 +299,43 @@ class MaskedAttention(Part):
         q = ws.alloc((T, self.nh * self.kw), torch.float32)
         table = ctx.page_table(cache.group)
         with ctx.prof("rotate_append"):
-            ops.rotate_append(qkv, bias, q, ctx.tok_pos, ctx.tok_seq, table, cache.k, cache.v, self.nh, self.nkv, self.kw, self.dv,
-                              self.rot, self.interleaved, self.freq, ctx.err, maps=self.maps, q_norm=self.q_norm, k_norm=self.k_norm,
-                              eps=float(self.qk_norm["eps"]) if self.qk_norm else 0.0,
-                              conv_w=self.conv_w if self.taps else None, conv_state=conv.state if conv is not None else None,
-                              seq_tok0=ctx.seq_tok0 if self.taps else None, seq_slot=ctx.seq_slots if self.taps else None, n_seqs=ctx.n_seqs,
-                              rot_mult=rotary_magnitude(self.rot_scaling))
+            if self.norm_all:
+                ops.norm_append(qkv, bias, q, ctx.tok_pos, ctx.tok_seq, table, cache.k, cache.v, self.nh, self.nkv, self.dk, self.dv, self.rot,
+                                self.interleaved, self.freq, ctx.err, self.q_norm, self.k_norm, float(self.qk_norm["eps"]),
+                                rot_mult=rotary_magnitude(self.rot_scaling))
+            else:
+                ops.rotate_append(qkv, bias, q, ctx.tok_pos, ctx.tok_seq, table, cache.k, cache.v, self.nh, self.nkv, self.kw, self.dv,
+                                  self.rot, self.interleaved, self.freq, ctx.err, maps=self.maps, q_norm=self.q_norm, k_norm=self.k_norm,
+                                  eps=float(self.qk_norm["eps"]) if self.qk_norm else 0.0,
+                                  conv_w=self.conv_w if self.taps else None, conv_state=conv.state if conv is not None else None,
+                                  seq_tok0=ctx.seq_tok0 if self.taps else None, seq_slot=ctx.seq_slots if self.taps else None, n_seqs=ctx.n_seqs,
+                                  rot_mult=rotary_magnitude(self.rot_scaling))
         a = ws.alloc((T, self.nh * self.maps * self.dv), torch.float32 if self.diff else self.dtype)
         with ctx.prof("attn_masked"):
             pairs = T * self.nh * self.maps
-            long_and_few = ctx.all_single and most_keys(self.mask, self.mask_size) > SPLIT_KEYS_FROM and pairs < 2 * ctx.n_sms
+            long_and_few = ctx.all_single and most_keys(self.mask, self.mask_size, self.keep) > SPLIT_KEYS_FROM and pairs < 2 * ctx.n_sms
             if ctx.all_single and (self.nh // self.nkv >= SHARED_KEYS_MIN_GROUP or (long_and_few and self.nh // self.nkv >= SHARED_KEYS_LONG_GROUP)):
-                splits = decode_splits(ctx, self.nkv * self.maps, self.nh // self.nkv, self.mask, self.mask_size)
+                splits = decode_splits(ctx, self.nkv * self.maps, self.nh // self.nkv, self.mask, self.mask_size, self.keep)
                 part = ws.alloc((T * self.nh * self.maps * splits * (2 + self.dv),), torch.float32) if splits > 1 else None
                 tseq, ttok0, tntok, tpos0 = single_token_tiles(ctx)
                 ops.masked_attn_tiled(q, a, cache.k, cache.v, table, tseq, ttok0, tntok, tpos0, T, 1, self.nh, self.nkv, self.dk, self.dv,
-                                      self.scale, self.mask, self.mask_size, self.sink, n_splits=splits, part=part, maps=self.maps, gate=gate)
+                                      self.scale, self.mask, self.mask_size, self.sink, n_splits=splits, part=part, maps=self.maps, gate=gate, keep=self.keep)
             elif ctx.all_single:
-                splits = head_splits(ctx, T * self.nh * self.maps, self.mask, self.mask_size)
+                splits = head_splits(ctx, T * self.nh * self.maps, self.mask, self.mask_size, self.keep)
                 part = ws.alloc((T * self.nh * self.maps * splits * (2 + self.dv),), torch.float32) if splits > 1 else None
                 ops.masked_attn(q, a, cache.k, cache.v, ctx.tok_pos, ctx.tok_seq, table, self.nh, self.nkv, self.dk, self.dv, self.scale,
-                                self.mask, self.mask_size, self.sink, most_keys(self.mask, self.mask_size), maps=self.maps, gate=gate,
-                                n_splits=splits, part=part)
+                                self.mask, self.mask_size, self.sink, most_keys(self.mask, self.mask_size, self.keep), maps=self.maps, gate=gate,
+                                n_splits=splits, part=part, keep=self.keep)
             elif self._on_tensor_cores():
                 tiles = ctx.tiles(ops.SPLIT_PREFILL_TILE)
                 ops.attn_prefill_split(q, a, cache.k, cache.v, table, tiles.seq, tiles.tok0, tiles.ntok, tiles.pos0, tiles.count, self.nh, self.nkv,
-                                       self.dk, self.dv, self.scale, gate=gate, mask=self.mask, mask_size=self.mask_size, sink=self.sink,
+                                       self.dk, self.dv, self.scale, gate=gate, mask=self.mask, mask_size=self.mask_size, sink=self.sink, keep=self.keep,
                                        max_keys=max(p + n for p, n in zip(ctx.seq_first_positions, ctx.seq_lengths)))
             else:
                 tiles = ctx.tiles(self.tile_tokens)
                 ops.masked_attn_tiled(q, a, cache.k, cache.v, table, tiles.seq, tiles.tok0, tiles.ntok, tiles.pos0, tiles.count,
                                       self.tile_tokens, self.nh, self.nkv, self.dk, self.dv, self.scale, self.mask, self.mask_size, self.sink,
-                                      maps=self.maps, gate=gate)
+                                      maps=self.maps, gate=gate, keep=self.keep)
         if self.diff:
             o = ws.alloc((T, self.nh * self.dv), self.dtype)
             with ctx.prof("diff_combine"):

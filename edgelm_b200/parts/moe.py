@@ -13,7 +13,7 @@ Options, each with its constants in the spec:
     router    {"kind": "scored", ...}: scores s = softmax(z) over ALL experts, or with `score` "sigmoid" each expert's sigmoid(z);
               the choice takes the `top` largest of s + a correction per expert (a tensor, `names["correction"]`, if the names have
               it), looking only inside the `keep` of `groups` equal groups
-              of neighbouring experts whose largest corrected score is largest (other experts count as minus infinity: if the
+              of neighbouring experts whose largest corrected score (`group_score` "top2_sum": the sum of whose two largest) is largest (other experts count as minus infinity: if the
               kept groups hold fewer than `top` experts, the others follow in the order of their numbers);
               the weights are the chosen experts' s over their sum (+ 1e-20) (`renormalize` False: s as it is), times `scale`.  `identity`: so many router
               outputs after the experts' belong to identity experts, which have no tensors and return their input (they
@@ -47,6 +47,9 @@ class MixtureOfExperts(Part):
         if self.router not in ("top_logits", "scored"):
             raise ConfigError(f"moe: a router of kind '{self.router}' is not known (top_logits, scored)")
         self.score, self.renormalize = r.get("score", "softmax"), bool(r.get("renormalize", True))
+        self.group_score = r.get("group_score", "max")
+        if self.group_score not in ops.GROUP_SCORES:
+            raise ConfigError(f"moe: a group score '{self.group_score}' is not known ({', '.join(ops.GROUP_SCORES)})")
         if self.score not in ops.ROUTER_SCORES or (self.router != "scored" and (self.score, self.renormalize) != ("softmax", True)):
             raise ConfigError(f"moe: a router of kind '{self.router}' with score '{self.score}' is not known")
         self.weight_on = spec.get("weight_on", "output")
@@ -72,6 +75,8 @@ class MixtureOfExperts(Part):
         if self.router == "scored":
             out.update({"router": "scored", "identity_experts": self.identity, "expert_groups": self.groups, "groups_kept": self.keep,
                         "router_scale": self.scale, "router_score": self.score})
+            if self.groups > 1 and self.group_score != "max":
+                out["group_score"] = self.group_score
         if self.weight_on == "input":
             out["weight_on"] = "input"
         if self.glu != tuple(ops.GLU_SWIGLU):
@@ -143,7 +148,13 @@ class MixtureOfExperts(Part):
     def first_weights(self):
         return ()
 
-    def forward(self, ctx, h, x, accumulate=True):
+    def takes_norm(self, norm):
+        """Whether `forward(..., norm=norm)` is open: the norm on the sublayer's output in the same pass as the experts' weighted sum."""
+        return norm.kind == "rmsnorm" and not self.identity and not self.shared_gate
+
+    def forward(self, ctx, h, x, accumulate=True, norm=None, cast=None):
+        """x += feed_forward(h), or with `accumulate` False x = feed_forward(h); with `norm` (see `takes_norm`) x += norm(feed_forward(h)),
+        and `cast` (optional) receives the new x in the compute dtype."""
         h = linear.as_tensor(h)
         T, ws = h.shape[0], ctx.ws
         tc = self._on_tensor_cores()
@@ -159,7 +170,7 @@ class MixtureOfExperts(Part):
         with ctx.prof("moe_route"):
             if self.router == "scored":
                 ops.moe_route_scored(h, self.w_router, self.correction, idx, wts, self.top, self.routed, self.groups, self.keep, self.scale, extra=gate,
-                                     score=self.score, renormalize=self.renormalize)
+                                     score=self.score, renormalize=self.renormalize, group_score=self.group_score)
             else:
                 ops.moe_route(h, self.w_router, self.b_router, idx, wts, self.top)
             ops.moe_plan(idx, self.n_experts, tile_rows, row_pair, pair_row, tile_expert)     # (an identity expert's pair gets no row)
@@ -181,14 +192,18 @@ class MixtureOfExperts(Part):
             with ctx.prof("moe_down"):
                 ops.moe_down(mid, self.w_down, y, row_pair, tile_expert, self.top)
         ys = None
-        if self.shared is not None and not self.shared_gate:      # (nothing to multiply by: straight into x, in its last product's epilogue)
-            with ws.frame():
-                self.shared.forward(ctx, h, x, accumulate=accumulate)
-            accumulate = True
-        elif self.shared is not None:
+        if self.shared is not None and (self.shared_gate or norm is not None):
             ys = ws.alloc((T, self.hidden), torch.float32)
             with ws.frame():
                 self.shared.forward(ctx, h, ys, accumulate=False)
+        elif self.shared is not None:      # (nothing to multiply by: straight into x, in its last product's epilogue)
+            with ws.frame():
+                self.shared.forward(ctx, h, x, accumulate=accumulate)
+            accumulate = True
+        if norm is not None:
+            with ctx.prof("moe_combine"):
+                ops.moe_combine_norm(x, y, wts if in_weight is None else None, pair_row, norm.weight, norm.eps, shared=ys, cast=cast, top=self.top)
+            return
         with ctx.prof("moe_combine"):
             if not accumulate:
                 x.zero_()
