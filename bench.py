@@ -8,6 +8,7 @@
     python bench.py --design redenex        # the same for the Redenex design
     python bench.py --design radupel        # the Radupel design beside the Sagizen design at equal sizes
     python bench.py --design sarizen        # the Sarizen design beside the Vosulorn and the Radupel designs at equal sizes
+    python bench.py --design semadra        # the Semadra design beside the Sarizen and the Vosulorn designs at equal sizes
 
 A "step" is one decode step of the whole batch.  The default run has the layer sizes of the
 SmolLM2-135M-shaped configuration with random weights N(0, 0.02), bfloat16, a batch of 8
@@ -269,7 +270,9 @@ DESIGN_PAIRS = {"sagizen": [("sagizen-576", "smollm2-135m", 8), ("sagizen-2048",
                 # (the closest earlier model: the design whose layers also hold an attention beside a linear recurrence)
                 "radupel": [("radupel-576", "sagizen-576", 8), ("radupel-2048", "sagizen-2048", 4)],
                 # (two earlier models share its parts: latent attention and experts; linear attention, experts and the layers' arrangement)
-                "sarizen": [("sarizen-576", "vosulorn-576", 8), ("sarizen-2048", "vosulorn-2048", 4), ("sarizen-2048", "radupel-2048", 4)]}
+                "sarizen": [("sarizen-576", "vosulorn-576", 8), ("sarizen-2048", "vosulorn-2048", 4), ("sarizen-2048", "radupel-2048", 4)],
+                # (windowed latent attention, sigmoid-scored and shared experts; attention under a mask beside latent attention)
+                "semadra": [("semadra-576", "sarizen-576", 8), ("semadra-2048", "sarizen-2048", 4), ("semadra-2048", "vosulorn-2048", 4)]}
 
 
 def parts_profile(model, vocab, ctx, prompt_tokens=2048, batch=8):

@@ -163,11 +163,7 @@ rotate_append_kernel(const float* __restrict__ qkv, const float* __restrict__ bi
 // `k_norm` [G dk], before they are split into heads; then the rotation (`rot` dimensions of every head, 0: none) and the cache.
 // A block a token; the row lies in shared memory between its sums of squares and the scaling.  V: values a thread takes at a
 // time (4: dk, dv and the rows' pitch are multiples of 4 and everything is aligned).
-__device__ __forceinline__ void store_values(float* dst, const float (&x)[4]) { *reinterpret_cast<float4*>(dst) = make_float4(x[0], x[1], x[2], x[3]); }
-__device__ __forceinline__ void store_values(__nv_bfloat16* dst, const float (&x)[4]) {
-  const __nv_bfloat162 lo = __floats2bfloat162_rn(x[0], x[1]), hi = __floats2bfloat162_rn(x[2], x[3]);
-  *reinterpret_cast<uint2*>(dst) = make_uint2(*reinterpret_cast<const uint32_t*>(&lo), *reinterpret_cast<const uint32_t*>(&hi));
-}
+template <typename T> __device__ __forceinline__ void store_values(T* dst, const float (&x)[4]) { store_piece(dst, make_float4(x[0], x[1], x[2], x[3])); }
 template <typename T> __device__ __forceinline__ void store_values(T* dst, const float (&x)[1]) { *dst = from_f32<T>(x[0]); }
 
 template <typename T, int V>
@@ -180,7 +176,7 @@ norm_append_kernel(const float* __restrict__ qkv, const float* __restrict__ bias
   pdl_launch_dependents();
   pdl_wait();
   extern __shared__ __align__(16) float na_row[];      // (H + G) dk values
-  __shared__ float red[33];
+  __shared__ float red[66];
   const int t = blockIdx.x, pos = tok_pos[t];
   if (pos < 0) {
     if (threadIdx.x == 0) atomicOr(err, ERR_POSITION_RANGE);
@@ -208,8 +204,7 @@ norm_append_kernel(const float* __restrict__ qkv, const float* __restrict__ bias
     if (i < nq) sq += ss;
     else sk += ss;
   }
-  sq = block_sum(sq, red);
-  sk = block_sum(sk, red);
+  block_sum2(sq, sk, red);
   const float iq = 1.0f / sqrtf(sq / (float)nq + eps), ik = 1.0f / sqrtf(sk / (float)(G * dk) + eps);
   if (rot > 0) {      // (a rotated value needs its partner's norm too: the row is scaled in place first)
     for (int i = threadIdx.x; i < nqk; i += blockDim.x) na_row[i] *= i < nq ? iq * q_norm[i] : ik * k_norm[i - nq];
@@ -246,7 +241,7 @@ norm_append_kernel(const float* __restrict__ qkv, const float* __restrict__ bias
 // latent of the queries: divided by its root mean square (eps), times `ql_w`, row t of ql_out in the cache's type (the input of
 // the product that makes the queries).
 template <typename T>
-__global__ void __launch_bounds__(256)
+__global__ void __launch_bounds__(1024)
 latent_prepare_kernel(const float* __restrict__ u, int ldu, int kv_off, int has_kv, float* __restrict__ q_out, int q_pitch, int q_off,
                       int copy_q, const float* __restrict__ norm_w, float eps, const int32_t* __restrict__ tok_pos,
                       const int32_t* __restrict__ tok_seq, const int32_t* __restrict__ page_table, int table_stride, int n_pages,
@@ -255,7 +250,7 @@ latent_prepare_kernel(const float* __restrict__ u, int ldu, int kv_off, int has_
                       T* __restrict__ ql_out) {
   pdl_launch_dependents();
   pdl_wait();
-  __shared__ float red[33];
+  __shared__ float red[66];
   const int t = blockIdx.x;
   const int pos = tok_pos[t];
   if (pos < 0) {
@@ -273,13 +268,17 @@ latent_prepare_kernel(const float* __restrict__ u, int ldu, int kv_off, int has_
       const int h = i / d, j = i - h * d;
       qo[(size_t)h * q_pitch + j] = row[(size_t)h * (d + rd) + j];
     }
+  const float* cq = row + ql_off;
+  const float* c = row + kv_off;
+  float sq = 0.f, ss = 0.f;
+  if (ql_out)
+    for (int i = threadIdx.x; i < ql_rank; i += blockDim.x) sq = fmaf(cq[i], cq[i], sq);
+  if (has_kv)
+    for (int i = threadIdx.x; i < r; i += blockDim.x) ss = fmaf(c[i], c[i], ss);
+  block_sum2(sq, ss, red);
   if (ql_out) {
-    const float* c = row + ql_off;
-    float ss = 0.f;
-    for (int i = threadIdx.x; i < ql_rank; i += blockDim.x) ss = fmaf(c[i], c[i], ss);
-    ss = block_sum(ss, red);
-    const float inv = 1.0f / sqrtf(ss / (float)ql_rank + eps);
-    for (int i = threadIdx.x; i < ql_rank; i += blockDim.x) ql_out[(size_t)t * ql_rank + i] = from_f32<T>(c[i] * inv * ql_w[i]);
+    const float inv = 1.0f / sqrtf(sq / (float)ql_rank + eps);
+    for (int i = threadIdx.x; i < ql_rank; i += blockDim.x) ql_out[(size_t)t * ql_rank + i] = from_f32<T>(cq[i] * inv * ql_w[i]);
   }
   if (!has_kv) return;
   const int page = page_table[(size_t)tok_seq[t] * table_stride + pos / PAGE];
@@ -287,10 +286,6 @@ latent_prepare_kernel(const float* __restrict__ u, int ldu, int kv_off, int has_
     if (threadIdx.x == 0) atomicOr(err, ERR_PAGE_RANGE);
     return;
   }
-  const float* c = row + kv_off;
-  float ss = 0.f;
-  for (int i = threadIdx.x; i < r; i += blockDim.x) ss = fmaf(c[i], c[i], ss);
-  ss = block_sum(ss, red);
   const float inv = 1.0f / sqrtf(ss / (float)r + eps);
   T* dst = kcache + ((size_t)page * PAGE + pos % PAGE) * (r + rd);
   T* dst2 = row_out ? row_out + (size_t)t * (r + rd) : nullptr;
@@ -540,6 +535,116 @@ masked_attn_kernel(const float* __restrict__ q, TO* __restrict__ out, const T* _
   }
 }
 
+// The same for bfloat16 heads of at most 8 LK and 8 LV dimensions (multiples of 8), with a key row and a value row shared by LK and LV
+// lanes, 16 bytes each: a warp's loads are whole rows one after the other, and a chunk's 32 keys and 32 values are all requested
+// before the first is used.  Partial scores are added over the lanes of a row; each lane's weighted values over the warp's rows at the end.
+template <int LK, int LV>
+__global__ void __launch_bounds__(MA_MAX_WARPS * 32)
+masked_attn_rows_kernel(const float* __restrict__ q, __nv_bfloat16* __restrict__ out, const __nv_bfloat16* __restrict__ kcache,
+                        const __nv_bfloat16* __restrict__ vcache, const int32_t* __restrict__ tok_pos, const int32_t* __restrict__ tok_seq,
+                        const int32_t* __restrict__ page_table, int table_stride, int n_pages, int H, int G, int dk, int dv, float scale, int mask,
+                        int mask_size, const float* __restrict__ sink, const float* __restrict__ gate, int ldg, int n_splits,
+                        float* __restrict__ part, int keep, int gate_ch) {
+  constexpr int KPS = 32 / LK, VPS = 32 / LV;      // keys and values that a warp's load covers
+  pdl_launch_dependents();
+  pdl_wait();
+  extern __shared__ __align__(16) float ma_smem[];
+  const int t = blockIdx.x, h = blockIdx.y, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, NW = blockDim.x >> 5;
+  float* wm = ma_smem;
+  float* wl = wm + NW;
+  float* wo = wl + NW;             // [NW][dv]
+  const int pos = tok_pos[t];
+  if (pos < 0) return;
+  const int g = h / (H / G);
+  const int32_t* table = page_table + (size_t)tok_seq[t] * table_stride;
+  const int kd = (lane % LK) * 8, vd = (lane % LV) * 8;       // this lane's dimensions of a row
+  float qv[8];
+#pragma unroll
+  for (int j = 0; j < 8; ++j) qv[j] = kd < dk ? q[((size_t)t * H + h) * dk + kd + j] * scale : 0.f;
+  const int lo = first_key(pos, mask, mask_size), kept = min(keep, lo), n_keys = kept + pos - lo + 1;
+  const int n_chunks = (n_keys + 31) >> 5, per_split = (n_chunks + n_splits - 1) / n_splits;
+  const int c_end = min(n_chunks, ((int)blockIdx.z + 1) * per_split);
+  float m = -INFINITY, l = 0.f, o[8] = {};
+  for (int c = blockIdx.z * per_split + warp; c < c_end; c += NW) {
+    int row = -1;                  // the row of key c * 32 + lane
+    if (c * 32 + lane < n_keys) {
+      const int i = c * 32 + lane, p = i < kept ? i : lo + i - kept, page = table[p / PAGE];
+      if (page >= 0 && page < n_pages) row = (page * G + g) * PAGE + p % PAGE;
+    }
+    uint4 kr[LK], vr[LV];
+#pragma unroll
+    for (int s = 0; s < LK; ++s) {
+      const int r = __shfl_sync(0xffffffffu, row, s * KPS + lane / LK);
+      kr[s] = r >= 0 && kd < dk ? *reinterpret_cast<const uint4*>(kcache + (size_t)r * dk + kd) : make_uint4(0u, 0u, 0u, 0u);
+    }
+#pragma unroll
+    for (int s = 0; s < LV; ++s) {
+      const int r = __shfl_sync(0xffffffffu, row, s * VPS + lane / LV);
+      vr[s] = r >= 0 && vd < dv ? *reinterpret_cast<const uint4*>(vcache + (size_t)r * dv + vd) : make_uint4(0u, 0u, 0u, 0u);
+    }
+    float sc = -INFINITY;
+#pragma unroll
+    for (int s = 0; s < LK; ++s) {
+      const uint4 k4 = kr[s];
+      float a = qv[0] * __uint_as_float(k4.x << 16), b = qv[1] * __uint_as_float(k4.x & 0xffff0000u);
+      a = fmaf(qv[2], __uint_as_float(k4.y << 16), a); b = fmaf(qv[3], __uint_as_float(k4.y & 0xffff0000u), b);
+      a = fmaf(qv[4], __uint_as_float(k4.z << 16), a); b = fmaf(qv[5], __uint_as_float(k4.z & 0xffff0000u), b);
+      a = fmaf(qv[6], __uint_as_float(k4.w << 16), a); b = fmaf(qv[7], __uint_as_float(k4.w & 0xffff0000u), b);
+      a += b;
+#pragma unroll
+      for (int x = LK / 2; x > 0; x >>= 1) a += __shfl_xor_sync(0xffffffffu, a, x);
+      const float mine = __shfl_sync(0xffffffffu, a, (lane % KPS) * LK);      // key s * KPS + j lies in the lanes from j * LK
+      if (lane / KPS == s) sc = mine;
+    }
+    if (row < 0) sc = -INFINITY;
+    const float m_new = fmaxf(m, warp_max(sc));
+    if (m_new == -INFINITY) continue;
+    const float w = sc == -INFINITY ? 0.f : expf(sc - m_new), corr = m == -INFINITY ? 0.f : expf(m - m_new);
+    l = l * corr + warp_sum(w);
+    m = m_new;
+#pragma unroll
+    for (int j = 0; j < 8; ++j) o[j] *= corr;
+#pragma unroll
+    for (int s = 0; s < LV; ++s) {
+      const float ws = __shfl_sync(0xffffffffu, w, s * VPS + lane / LV);
+      const uint4 v4 = vr[s];
+      o[0] = fmaf(ws, __uint_as_float(v4.x << 16), o[0]); o[1] = fmaf(ws, __uint_as_float(v4.x & 0xffff0000u), o[1]);
+      o[2] = fmaf(ws, __uint_as_float(v4.y << 16), o[2]); o[3] = fmaf(ws, __uint_as_float(v4.y & 0xffff0000u), o[3]);
+      o[4] = fmaf(ws, __uint_as_float(v4.z << 16), o[4]); o[5] = fmaf(ws, __uint_as_float(v4.z & 0xffff0000u), o[5]);
+      o[6] = fmaf(ws, __uint_as_float(v4.w << 16), o[6]); o[7] = fmaf(ws, __uint_as_float(v4.w & 0xffff0000u), o[7]);
+    }
+  }
+#pragma unroll
+  for (int j = 0; j < 8; ++j)
+#pragma unroll
+    for (int x = LV; x < 32; x <<= 1) o[j] += __shfl_xor_sync(0xffffffffu, o[j], x);
+  if (lane == 0) { wm[warp] = m; wl[warp] = l; }
+  if (lane < LV && vd < dv)
+#pragma unroll
+    for (int j = 0; j < 8; ++j) wo[warp * dv + vd + j] = o[j];
+  __syncthreads();
+  float M = n_splits == 1 && sink ? sink[h] : -INFINITY;
+  for (int w2 = 0; w2 < NW; ++w2) M = fmaxf(M, wm[w2]);
+  float L = n_splits == 1 && sink ? expf(sink[h] - M) : 0.f;
+  for (int w2 = 0; w2 < NW; ++w2) L += wm[w2] == -INFINITY ? 0.f : wl[w2] * expf(wm[w2] - M);
+  float* dst = n_splits > 1 ? part + (((size_t)t * H + h) * n_splits + blockIdx.z) * (2 + dv) : nullptr;
+  if (dst && threadIdx.x == 0) { dst[0] = M; dst[1] = L; }
+  float inv = L > 0.f ? 1.0f / L : 0.f;
+  const float* grow = gate ? gate + (size_t)t * ldg : nullptr;
+  if (gate && !gate_ch) inv *= gate_factor(grow, 0, h, 0);
+  for (int d = threadIdx.x; d < dv; d += blockDim.x) {
+    float acc = 0.f;
+    for (int w2 = 0; w2 < NW; ++w2)
+      if (wm[w2] != -INFINITY) acc = fmaf(wo[w2 * dv + d], expf(wm[w2] - M), acc);
+    if (dst) {
+      dst[2 + d] = acc;
+      continue;
+    }
+    if (gate && gate_ch) acc *= gate_factor(grow, gate_ch, h, d);
+    out[((size_t)t * H + h) * dv + d] = from_f32<__nv_bfloat16>(acc * inv);
+  }
+}
+
 // ---- prompt steps
 // A block = up to 32 (token, query head) rows of one key/value head and of one run of consecutive tokens (a tile of the
 // step's metadata); a page of 64 keys with their values is staged in shared memory as float32 once for all the rows.
@@ -755,23 +860,38 @@ __global__ void masked_attn_fold_kernel(const float* __restrict__ part, TO* __re
                                         int n_splits, const float* __restrict__ gate, int ldg, int maps, int gate_ch) {
   pdl_launch_dependents();
   pdl_wait();
-  const int t = blockIdx.x, h = blockIdx.y;
+  __shared__ float factor[64], denom;      // what a split's weighted values are multiplied by; the denominator of all of them
+  const int t = blockIdx.x, h = blockIdx.y, lane = threadIdx.x & 31;
   const float* p = part + ((size_t)t * H + h) * n_splits * (2 + dv);
-  float M = sink ? sink[h] : -INFINITY;
-  for (int s = 0; s < n_splits; ++s) M = fmaxf(M, p[(size_t)s * (2 + dv)]);
-  float L = sink ? expf(sink[h] - M) : 0.f;
-  for (int s = 0; s < n_splits; ++s) {
-    const float ms = p[(size_t)s * (2 + dv)];
-    if (ms != -INFINITY) L += p[(size_t)s * (2 + dv) + 1] * expf(ms - M);
+  if (threadIdx.x < 32) {
+    float m[2], l[2];
+#pragma unroll
+    for (int j = 0; j < 2; ++j) {
+      const int s = lane + 32 * j;
+      m[j] = s < n_splits ? p[(size_t)s * (2 + dv)] : -INFINITY;
+      l[j] = s < n_splits ? p[(size_t)s * (2 + dv) + 1] : 0.f;
+    }
+    const float M = fmaxf(warp_max(fmaxf(m[0], m[1])), sink ? sink[h] : -INFINITY);
+    float sum = 0.f;
+#pragma unroll
+    for (int j = 0; j < 2; ++j) {
+      const float f = m[j] != -INFINITY ? expf(m[j] - M) : 0.f;
+      if (lane + 32 * j < n_splits) factor[lane + 32 * j] = f;
+      sum = f > 0.f ? fmaf(l[j], f, sum) : sum;
+    }
+    sum = warp_sum(sum);
+    if (lane == 0) denom = sum + (sink ? expf(sink[h] - M) : 0.f);
   }
-  float inv = L > 0.f ? 1.0f / L : 0.f;
+  __syncthreads();
+  float inv = denom > 0.f ? 1.0f / denom : 0.f;
   const float* grow = gate ? gate + (size_t)t * ldg : nullptr;
   if (gate && !gate_ch) inv *= gate_factor(grow, 0, h / maps, 0);      // the head's output gate
   for (int d = threadIdx.x; d < dv; d += blockDim.x) {
     float acc = 0.f;
-    for (int s = 0; s < n_splits; ++s) {
-      const float ms = p[(size_t)s * (2 + dv)];
-      if (ms != -INFINITY) acc = fmaf(p[(size_t)s * (2 + dv) + 2 + d], expf(ms - M), acc);
+#pragma unroll 8
+    for (int s = 0; s < n_splits; ++s) {      // (a split that saw nothing left no values: its factor is 0, its memory is not read)
+      const float f = factor[s];
+      acc = f > 0.f ? fmaf(f, p[(size_t)s * (2 + dv) + 2 + d], acc) : acc;
     }
     if (gate && gate_ch) acc *= gate_factor(grow, gate_ch, h / maps, d);
     out[((size_t)t * H + h) * dv + d] = from_f32<TO>(acc * inv);
@@ -907,13 +1027,14 @@ extern "C" int edgelm_latent_prepare(const float* u, int ldu, int kv_off, int ha
   EL_REFUSE(rd == 0 || freq != nullptr, "latent_prepare: no frequencies");
   EL_REFUSE(H * (d + rd) <= ldu && (!has_kv || kv_off + r + rd <= ldu), "latent_prepare: rows of %d values are too short", ldu);
   EL_REFUSE(H == 0 || (q_off >= (copy_q ? d : 0) && q_off + rd <= q_pitch), "latent_prepare: a query head of %d values does not hold %d at %d", q_pitch, rd, q_off);
+  const int threads = n_tokens <= 64 ? 1024 : 256;      // (few tokens: a row is one trip to memory)
   const int bit = pdl_bit_for_tokens(n_tokens);
   if (dtype == DT_F32)
-    launch_pdl(bit, latent_prepare_kernel<float>, dim3(n_tokens), dim3(256), (size_t)0, stream, u, ldu, kv_off, has_kv, q_out, q_pitch, q_off, copy_q,
+    launch_pdl(bit, latent_prepare_kernel<float>, dim3(n_tokens), dim3(threads), (size_t)0, stream, u, ldu, kv_off, has_kv, q_out, q_pitch, q_off, copy_q,
                norm_w, eps, tok_pos, tok_seq, page_table, table_stride, n_pages, (float*)kcache, (float*)row_out, H, d, rd, r, freq, err, interleaved, mult,
                ql_off, ql_rank, ql_w, (float*)ql_out);
   else if (dtype == DT_BF16)
-    launch_pdl(bit, latent_prepare_kernel<__nv_bfloat16>, dim3(n_tokens), dim3(256), (size_t)0, stream, u, ldu, kv_off, has_kv, q_out, q_pitch, q_off,
+    launch_pdl(bit, latent_prepare_kernel<__nv_bfloat16>, dim3(n_tokens), dim3(threads), (size_t)0, stream, u, ldu, kv_off, has_kv, q_out, q_pitch, q_off,
                copy_q, norm_w, eps, tok_pos, tok_seq, page_table, table_stride, n_pages, (__nv_bfloat16*)kcache, (__nv_bfloat16*)row_out, H, d, rd,
                r, freq, err, interleaved, mult, ql_off, ql_rank, ql_w, (__nv_bfloat16*)ql_out);
   else
@@ -979,6 +1100,21 @@ static void launch_masked(const float* q, void* out, const void* kcache, const v
                           const int32_t* page_table, int table_stride, int n_pages, int n_tokens, int H, int G, int dk, int dv, float scale,
                           int mask, int mask_size, const float* sink, int warps, int maps, const float* gate, int ldg, int n_splits, float* part,
                           int keep, int gate_ch, cudaStream_t stream) {
+  if constexpr (sizeof(T) == 2 && sizeof(TO) == 2) {      // whole rows at a time, where the heads allow it
+    if (maps == 1 && vcache && dk % 8 == 0 && dv % 8 == 0 && dk <= 128 && dv <= 128 && (uintptr_t)kcache % 16 == 0 && (uintptr_t)vcache % 16 == 0) {
+      const size_t smem = (size_t)warps * (2 + dv) * sizeof(float);
+      const int bit = pdl_bit_for_tokens(n_tokens);
+#define EL_MR(LK, LV) launch_pdl(bit, masked_attn_rows_kernel<LK, LV>, dim3(n_tokens, H, n_splits), dim3(warps * 32), smem, stream, q, (__nv_bfloat16*)out, (const __nv_bfloat16*)kcache, \
+                                 (const __nv_bfloat16*)vcache, tok_pos, tok_seq, page_table, table_stride, n_pages, H, G, dk, dv, scale, mask, mask_size, sink, gate, ldg, n_splits, part, keep, gate_ch)
+      if (dk <= 64) { if (dv <= 64) EL_MR(8, 8); else EL_MR(8, 16); }
+      else { if (dv <= 64) EL_MR(16, 8); else EL_MR(16, 16); }
+#undef EL_MR
+      if (n_splits > 1 && cudaPeekAtLastError() == cudaSuccess)
+        launch_pdl(bit, masked_attn_fold_kernel<TO>, dim3(n_tokens, H), dim3(dv >= 256 ? 256 : (dv > 64 ? 128 : 64)), (size_t)0, stream, (const float*)part, (TO*)out, sink, H, dv,
+                   n_splits, gate, ldg, 1, gate_ch);
+      return;
+    }
+  }
   const T* vb = vcache ? (const T*)vcache : (const T*)kcache;
   const int ldv = vcache ? dv : dk;
   const int vec_k = (dk % (16 / (int)sizeof(T)) == 0) && ((uintptr_t)kcache % 16 == 0);
@@ -1049,6 +1185,20 @@ static int launch_masked_tiled(const float* q, void* out, const void* kcache, co
     launch_pdl(bit, masked_attn_fold_kernel<TO>, dim3(n_tokens, H * maps), dim3(dv >= 256 ? 256 : 128), (size_t)0, stream, (const float*)part, (TO*)out, sink,
                H * maps, dv, n_splits, gate, ldg, maps, gate_ch);
   }
+  return 0;
+}
+
+// The splits' partial results [tokens][H][n_splits][2 + dv] of `edgelm_latent_decode` merged: out [tokens][H][dv] in `out_dtype`
+extern "C" int edgelm_masked_attn_fold(const float* part, void* out, int out_dtype, const float* sink, int n_tokens, int H, int dv, int n_splits,
+                                       const float* gate, int ldg, cudaStream_t stream) {
+  if (n_tokens == 0) return 0;
+  EL_REFUSE(n_tokens > 0 && H > 0 && H <= 65535 && dv >= 1 && n_splits >= 1 && n_splits <= 64, "masked_attn_fold: bad sizes");
+  const dim3 grid(n_tokens, H), block(dv >= 256 ? 256 : 128);
+  const int bit = pdl_bit_for_tokens(n_tokens);
+  if (out_dtype == DT_F32) launch_pdl(bit, masked_attn_fold_kernel<float>, grid, block, (size_t)0, stream, part, (float*)out, sink, H, dv, n_splits, gate, ldg, 1, 0);
+  else if (out_dtype == DT_BF16) launch_pdl(bit, masked_attn_fold_kernel<__nv_bfloat16>, grid, block, (size_t)0, stream, part, (__nv_bfloat16*)out, sink, H, dv, n_splits, gate, ldg, 1, 0);
+  else EL_REFUSE(false, "masked_attn_fold: unknown dtype code %d", out_dtype);
+  EL_LAUNCH_CHECK("masked_attn_fold");
   return 0;
 }
 

@@ -23,7 +23,7 @@
 // Takes key head sizes 32, 64, 96, 128 over value head sizes of these that are not larger.
 #include <math_constants.h>
 
-#include "common.cuh"
+#include "mma_split.cuh"
 
 namespace edgelm {
 
@@ -38,37 +38,6 @@ __device__ __forceinline__ int sp_first_key(int pos, int mask, int size) {
 
 constexpr int SP_WARPS = 4;
 constexpr int SP_ROWS = 16 * SP_WARPS;  // new tokens per block
-
-__device__ __forceinline__ uint32_t sp_smem(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
-
-__device__ __forceinline__ void sp_mma(float* c, uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0, uint32_t b1) {
-  asm volatile(
-      "mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
-      : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
-      : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
-}
-__device__ __forceinline__ void sp_ldmatrix_x4(uint32_t addr, uint32_t& r0, uint32_t& r1, uint32_t& r2, uint32_t& r3) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(r0), "=r"(r1), "=r"(r2), "=r"(r3) : "r"(addr));
-}
-__device__ __forceinline__ void sp_ldmatrix_x4_trans(uint32_t addr, uint32_t& r0, uint32_t& r1, uint32_t& r2, uint32_t& r3) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(r0), "=r"(r1), "=r"(r2), "=r"(r3) : "r"(addr));
-}
-__device__ __forceinline__ void sp_cp16(uint32_t dst, const void* src, int src_bytes) {
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(src_bytes) : "memory");
-}
-
-// Two float32 values as three packed pairs of bfloat16 terms: x = t1 + t2 + t3 up to float32 rounding (each term the
-// rounding of what the terms before left over; the remainders are exact in float32).
-__device__ __forceinline__ void sp_split(float x, float y, uint32_t& t1, uint32_t& t2, uint32_t& t3) {
-  const __nv_bfloat16 x1 = __float2bfloat16_rn(x), y1 = __float2bfloat16_rn(y);
-  const float xr = x - __bfloat162float(x1), yr = y - __bfloat162float(y1);
-  const __nv_bfloat16 x2 = __float2bfloat16_rn(xr), y2 = __float2bfloat16_rn(yr);
-  const __nv_bfloat16 x3 = __float2bfloat16_rn(xr - __bfloat162float(x2)), y3 = __float2bfloat16_rn(yr - __bfloat162float(y2));
-  const __nv_bfloat162 p1 = __halves2bfloat162(x1, y1), p2 = __halves2bfloat162(x2, y2), p3 = __halves2bfloat162(x3, y3);
-  t1 = *reinterpret_cast<const uint32_t*>(&p1);
-  t2 = *reinterpret_cast<const uint32_t*>(&p2);
-  t3 = *reinterpret_cast<const uint32_t*>(&p3);
-}
 
 template <int HDT, int VDT, int NG>  // key and value head sizes / 16 (even); warp groups that share the pages of a tile
 __global__ void __launch_bounds__(SP_WARPS * 32 * NG)
@@ -326,21 +295,25 @@ attn_prefill_split_kernel(const float* __restrict__ q, int ldq, __nv_bfloat16* _
     if (rowA < ntok) invA *= 1.0f / (1.0f + expf(-gate[(size_t)(tok0 + rowA) * ldg + head]));
     if (rowB < ntok) invB *= 1.0f / (1.0f + expf(-gate[(size_t)(tok0 + rowB) * ldg + head]));
   }
+  if (gate != nullptr && gate_ch) {     // a gate per channel: all of a row's numbers are requested before the first is used
+    float ga[VD / 8][4];
+    const float* gA = gate + (size_t)(tok0 + min(rowA, ntok - 1)) * ldg + head * VD + tig * 2;
+    const float* gB = gate + (size_t)(tok0 + min(rowB, ntok - 1)) * ldg + head * VD + tig * 2;
+#pragma unroll
+    for (int dt = 0; dt < VD / 8; ++dt) {
+      ga[dt][0] = gA[dt * 8];
+      ga[dt][1] = gA[dt * 8 + 1];
+      ga[dt][2] = gB[dt * 8];
+      ga[dt][3] = gB[dt * 8 + 1];
+    }
+#pragma unroll
+    for (int dt = 0; dt < VD / 8; ++dt)
+#pragma unroll
+      for (int j = 0; j < 4; ++j) o[dt][j] *= 1.0f / (1.0f + expf(-ga[dt][j]));
+  }
 #pragma unroll
   for (int dt = 0; dt < VD / 8; ++dt) {
     const int d = head * VD + dt * 8 + tig * 2;
-    if (gate != nullptr && gate_ch) {     // a gate per channel
-      if (rowA < ntok) {
-        const float* ga = gate + (size_t)(tok0 + rowA) * ldg + d;
-        o[dt][0] *= 1.0f / (1.0f + expf(-ga[0]));
-        o[dt][1] *= 1.0f / (1.0f + expf(-ga[1]));
-      }
-      if (rowB < ntok) {
-        const float* gb = gate + (size_t)(tok0 + rowB) * ldg + d;
-        o[dt][2] *= 1.0f / (1.0f + expf(-gb[0]));
-        o[dt][3] *= 1.0f / (1.0f + expf(-gb[1]));
-      }
-    }
     if (rowA < ntok) {
       const __nv_bfloat162 v = __floats2bfloat162_rn(o[dt][0] * invA, o[dt][1] * invA);
       *reinterpret_cast<__nv_bfloat162*>(out + (size_t)(tok0 + rowA) * ldo + d) = v;

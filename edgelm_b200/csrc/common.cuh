@@ -45,6 +45,13 @@ template <typename T> __device__ __forceinline__ T from_f32(float v);
 template <> __device__ __forceinline__ float from_f32<float>(float v) { return v; }
 template <> __device__ __forceinline__ __nv_bfloat16 from_f32<__nv_bfloat16>(float v) { return __float2bfloat16_rn(v); }
 
+// four values to consecutive places (16- or 8-byte aligned)
+__device__ __forceinline__ void store_piece(float* dst, const float4& v) { *reinterpret_cast<float4*>(dst) = v; }
+__device__ __forceinline__ void store_piece(__nv_bfloat16* dst, const float4& v) {
+  const __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
+  *reinterpret_cast<uint2*>(dst) = make_uint2(*reinterpret_cast<const uint32_t*>(&lo), *reinterpret_cast<const uint32_t*>(&hi));
+}
+
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
@@ -71,6 +78,23 @@ __device__ __forceinline__ float block_sum(float v, float* red) {
   }
   __syncthreads();
   return red[32];
+}
+
+// Two sums at once, each in the order of `block_sum`.  `red` holds 66 floats.
+__device__ __forceinline__ void block_sum2(float& a, float& b, float* red) {
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarp = (blockDim.x + 31) >> 5;
+  a = warp_sum(a);
+  b = warp_sum(b);
+  __syncthreads();
+  if (lane == 0) { red[warp] = a; red[33 + warp] = b; }
+  __syncthreads();
+  if (warp < 2) {
+    const float t = warp_sum(lane < nwarp ? red[33 * warp + lane] : 0.f);
+    if (lane == 0) red[33 * warp + 32] = t;
+  }
+  __syncthreads();
+  a = red[32];
+  b = red[65];
 }
 
 // Programmatic dependent launch: a kernel launched with `launch_pdl` may start while the kernel before

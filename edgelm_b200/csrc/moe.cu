@@ -22,9 +22,9 @@ namespace edgelm {
 
 constexpr int MOE_MAX_EXPERTS = 1024;
 
-// The router's logits of one token into shared memory: z[e] = wr[e] . h (+ br[e]).  A block a token: its four warps share the
+// The router's logits of one token into shared memory: z[e] = wr[e] . h (+ br[e]).  A block a token: its warps share the
 // width, eight experts at a time (the token's row is read once for the eight, and a thread has eight independent sums and
-// several steps of loads in flight); the warps' sums are added in a fixed order.  `part`: 32 floats.
+// several steps of loads in flight); the warps' sums are added in a fixed order.  `part`: 8 floats a warp.
 template <typename TH>
 __device__ __forceinline__ void moe_logits(const TH* __restrict__ row, const float* __restrict__ wr, const float* __restrict__ br,
                                            float* z, float* part, int D, int E) {
@@ -35,7 +35,7 @@ __device__ __forceinline__ void moe_logits(const TH* __restrict__ row, const flo
     for (int j = 0; j < 8; ++j) w[j] = wr + (size_t)min(e0 + j, E - 1) * D;     // (past the last expert: computed, not kept)
     float acc[8] = {};
 #pragma unroll 4
-    for (int i = threadIdx.x; i < D; i += 128) {
+    for (int i = threadIdx.x; i < D; i += blockDim.x) {
       const float x = to_f32(row[i]);
 #pragma unroll
       for (int j = 0; j < 8; ++j) acc[j] = fmaf(x, w[j][i], acc[j]);
@@ -46,20 +46,22 @@ __device__ __forceinline__ void moe_logits(const TH* __restrict__ row, const flo
       if (lane == 0) part[warp * 8 + j] = sj;
     }
     __syncthreads();
-    if (threadIdx.x < 8 && e0 + threadIdx.x < E)
-      z[e0 + threadIdx.x] = ((part[threadIdx.x] + part[8 + threadIdx.x]) + (part[16 + threadIdx.x] + part[24 + threadIdx.x])) +
-                            (br ? br[e0 + threadIdx.x] : 0.f);
+    if (threadIdx.x < 8 && e0 + threadIdx.x < E) {
+      float s = 0.f;
+      for (int w = 0; w < (int)(blockDim.x >> 5); ++w) s += part[w * 8 + threadIdx.x];
+      z[e0 + threadIdx.x] = s + (br ? br[e0 + threadIdx.x] : 0.f);
+    }
     __syncthreads();
   }
 }
 
 template <typename TH>
-__global__ void __launch_bounds__(128)
+__global__ void __launch_bounds__(512)
 moe_route_kernel(const TH* __restrict__ h, const float* __restrict__ wr, const float* __restrict__ br, int32_t* __restrict__ idx,
                  float* __restrict__ wts, int n_tokens, int D, int E, int top) {
   pdl_launch_dependents();
   pdl_wait();
-  extern __shared__ float mr_smem[];         // [E] logits, then [4][8] partial sums
+  extern __shared__ float mr_smem[];         // [E] logits, then [warps][8] partial sums
   float* z = mr_smem;
   moe_logits(h + (size_t)blockIdx.x * D, wr, br, z, mr_smem + E, D, E);
   const int t = blockIdx.x;
@@ -88,13 +90,13 @@ enum : int { SCORE_SOFTMAX = 0, SCORE_SIGMOID = 1 };
 // The scored router (see the head of this file).  E experts in all (the last ones may be identity experts: nothing here
 // treats them differently), `n_extra` more router rows whose sigmoid goes to extra[t][.].  Ties: the first of equal scores.
 template <typename TH>
-__global__ void __launch_bounds__(128)
+__global__ void __launch_bounds__(512)
 moe_route_scored_kernel(const TH* __restrict__ h, const float* __restrict__ wr, const float* __restrict__ correction,
                         int32_t* __restrict__ idx, float* __restrict__ wts, float* __restrict__ extra, int D, int E, int n_extra, int top,
                         int groups, int keep, float scale, int score, int renormalize, int group_top) {
   pdl_launch_dependents();
   pdl_wait();
-  extern __shared__ float mr_smem[];         // [E + n_extra] logits, [E] choice scores, [groups] group scores, then [4][8] partial sums
+  extern __shared__ float mr_smem[];         // [E + n_extra] logits, [E] choice scores, [groups] group scores, then [warps][8] partial sums
   float* z = mr_smem;
   float* c = z + E + n_extra;
   float* gs = c + E;
@@ -365,6 +367,66 @@ __global__ void moe_combine_norm_kernel(float* __restrict__ x, const float* __re
   }
 }
 
+// The same for rows of whole 16-byte pieces, up to MAXV of them a thread: the sum stays in registers
+template <typename TC, int MAXV>
+__global__ void __launch_bounds__(1024)
+moe_combine_norm_vec_kernel(float* __restrict__ x, const float* __restrict__ y, int ldy, const float* __restrict__ wts,
+                            const int32_t* __restrict__ pair_row, int top, int D, const float* __restrict__ shared, const float* __restrict__ w,
+                            float eps, TC* __restrict__ xc) {
+  pdl_launch_dependents();
+  __shared__ float red[33];
+  const int t = blockIdx.x, pieces = D >> 2;
+  float4 g[MAXV], v[MAXV], xv[MAXV];
+#pragma unroll
+  for (int j = 0; j < MAXV; ++j) {
+    const int i = threadIdx.x + j * blockDim.x;
+    if (i < pieces) g[j] = reinterpret_cast<const float4*>(w)[i];
+  }
+  pdl_wait();
+  const size_t row = (size_t)t * D;
+#pragma unroll
+  for (int j = 0; j < MAXV; ++j) {
+    const int i = threadIdx.x + j * blockDim.x;
+    v[j] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (i < pieces) xv[j] = reinterpret_cast<const float4*>(x + row)[i];
+  }
+#pragma unroll 4
+  for (int k = 0; k < top; ++k) {
+    const int r = pair_row[(size_t)t * top + k];
+    if (r < 0) continue;
+    const float wk = wts ? wts[(size_t)t * top + k] : 1.0f;
+    const float4* src = reinterpret_cast<const float4*>(y + (size_t)r * ldy);
+#pragma unroll
+    for (int j = 0; j < MAXV; ++j) {
+      const int i = threadIdx.x + j * blockDim.x;
+      if (i >= pieces) continue;
+      const float4 u = src[i];
+      v[j].x = fmaf(wk, u.x, v[j].x); v[j].y = fmaf(wk, u.y, v[j].y); v[j].z = fmaf(wk, u.z, v[j].z); v[j].w = fmaf(wk, u.w, v[j].w);
+    }
+  }
+  float ss = 0.f;
+#pragma unroll
+  for (int j = 0; j < MAXV; ++j) {
+    const int i = threadIdx.x + j * blockDim.x;
+    if (i >= pieces) continue;
+    if (shared) {
+      const float4 u = reinterpret_cast<const float4*>(shared + row)[i];
+      v[j].x += u.x; v[j].y += u.y; v[j].z += u.z; v[j].w += u.w;
+    }
+    ss = fmaf(v[j].x, v[j].x, ss); ss = fmaf(v[j].y, v[j].y, ss); ss = fmaf(v[j].z, v[j].z, ss); ss = fmaf(v[j].w, v[j].w, ss);
+  }
+  ss = block_sum(ss, red);
+  const float inv = 1.0f / sqrtf(ss / (float)D + eps);
+#pragma unroll
+  for (int j = 0; j < MAXV; ++j) {
+    const int i = threadIdx.x + j * blockDim.x;
+    if (i >= pieces) continue;
+    const float4 n = make_float4(xv[j].x + v[j].x * inv * g[j].x, xv[j].y + v[j].y * inv * g[j].y, xv[j].z + v[j].z * inv * g[j].z, xv[j].w + v[j].w * inv * g[j].w);
+    reinterpret_cast<float4*>(x + row)[i] = n;
+    if (xc) store_piece(xc + row + 4 * i, n);
+  }
+}
+
 }  // namespace edgelm
 
 using namespace edgelm;
@@ -373,6 +435,21 @@ extern "C" int edgelm_moe_combine_norm(float* x, const float* y, int ldy, const 
                                        const float* shared, const float* w, float eps, void* xc, int cast_dtype, cudaStream_t stream) {
   if (n_tokens == 0) return 0;
   EL_REFUSE(n_tokens > 0 && top >= 1 && D > 0 && ldy >= D && w != nullptr, "moe_combine_norm: bad sizes");
+  const bool vec = D % 4 == 0 && D <= 16384 && ldy % 4 == 0 && (uintptr_t)x % 16 == 0 && (uintptr_t)y % 16 == 0 && (uintptr_t)shared % 16 == 0 &&
+                   (uintptr_t)w % 16 == 0 && (uintptr_t)xc % 16 == 0;
+  if (vec) {
+    const int pieces = D / 4, most = n_tokens <= 64 ? 1024 : (pieces <= 2048 ? 256 : 512), threads = pieces < most ? (pieces + 31) / 32 * 32 : most;
+    const int per = (pieces + threads - 1) / threads, pb = pdl_bit_for_tokens(n_tokens);
+#define EL_CV(TC, V) launch_pdl(pb, moe_combine_norm_vec_kernel<TC, V>, dim3(n_tokens), dim3(threads), (size_t)0, stream, x, y, ldy, wts, pair_row, top, D, shared, w, eps, (TC*)xc)
+#define EL_CVV(TC) do { if (per <= 1) EL_CV(TC, 1); else if (per <= 2) EL_CV(TC, 2); else if (per <= 4) EL_CV(TC, 4); else EL_CV(TC, 8); } while (0)
+    if (xc == nullptr || cast_dtype == DT_F32) EL_CVV(float);
+    else if (cast_dtype == DT_BF16) EL_CVV(__nv_bfloat16);
+    else EL_REFUSE(false, "moe_combine_norm: unknown dtype code %d", cast_dtype);
+#undef EL_CVV
+#undef EL_CV
+    EL_LAUNCH_CHECK("moe_combine_norm");
+    return 0;
+  }
   const size_t smem = (size_t)D * sizeof(float);
   EL_REFUSE(smem <= 200 * 1024, "moe_combine_norm: rows of %d values", D);
   const dim3 grid(n_tokens), block(D >= 1024 ? (n_tokens <= 64 ? 1024 : 256) : 128);
@@ -388,14 +465,17 @@ extern "C" int edgelm_moe_combine_norm(float* x, const float* y, int ldy, const 
   return 0;
 }
 
+// Threads of a router's block: with few tokens enough for the row to be a trip or two to memory
+static int route_threads(int n_tokens, int D) { return n_tokens <= 64 && D >= 1024 ? 512 : 128; }
+
 extern "C" int edgelm_moe_tile_rows() { return MG_TM; }
 
 extern "C" int edgelm_moe_route(const void* h, int dtype, const float* wr, const float* br, int32_t* idx, float* wts, int n_tokens, int D,
                                 int E, int top, cudaStream_t stream) {
   if (n_tokens == 0) return 0;
   EL_REFUSE(n_tokens > 0 && D > 0 && E >= 1 && E <= MOE_MAX_EXPERTS && top >= 1 && top <= E, "moe_route: %d experts, %d chosen", E, top);
-  const dim3 grid(n_tokens), block(128);
-  const size_t smem = (size_t)(E + 32) * sizeof(float);
+  const dim3 grid(n_tokens), block(route_threads(n_tokens, D));
+  const size_t smem = (size_t)(E + block.x / 4) * sizeof(float);
   const int bit = pdl_bit_for_tokens(n_tokens);
   if (dtype == DT_F32) launch_pdl(bit, moe_route_kernel<float>, grid, block, smem, stream, (const float*)h, wr, br, idx, wts, n_tokens, D, E, top);
   else if (dtype == DT_BF16) launch_pdl(bit, moe_route_kernel<__nv_bfloat16>, grid, block, smem, stream, (const __nv_bfloat16*)h, wr, br, idx, wts, n_tokens, D, E, top);
@@ -413,8 +493,8 @@ extern "C" int edgelm_moe_route_scored(const void* h, int dtype, const float* wr
   EL_REFUSE(group_top == 1 || group_top == 2, "moe_route_scored: a group's worth from its %d largest scores", group_top);
   EL_REFUSE(n_extra >= 0 && n_extra <= 32 && (n_extra == 0 || extra != nullptr), "moe_route_scored: %d extra rows (up to 32)", n_extra);
   EL_REFUSE(score == SCORE_SOFTMAX || score == SCORE_SIGMOID, "moe_route_scored: unknown score %d", score);
-  const dim3 grid(n_tokens), block(128);
-  const size_t smem = (size_t)(2 * E + n_extra + groups + 32) * sizeof(float);
+  const dim3 grid(n_tokens), block(route_threads(n_tokens, D));
+  const size_t smem = (size_t)(2 * E + n_extra + groups + block.x / 4) * sizeof(float);
   const int bit = pdl_bit_for_tokens(n_tokens);
   if (dtype == DT_F32) launch_pdl(bit, moe_route_scored_kernel<float>, grid, block, smem, stream, (const float*)h, wr, correction, idx, wts, extra, D, E, n_extra, top, groups, keep, scale, score, renormalize, group_top);
   else if (dtype == DT_BF16) launch_pdl(bit, moe_route_scored_kernel<__nv_bfloat16>, grid, block, smem, stream, (const __nv_bfloat16*)h, wr, correction, idx, wts, extra, D, E, n_extra, top, groups, keep, scale, score, renormalize, group_top);

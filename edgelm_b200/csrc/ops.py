@@ -790,7 +790,12 @@ def head_matmul(a, a_head_stride, w, out, out_head_stride):
     _f32_rows(a, "a")
     _need(w.dim() == 3 and w.is_contiguous() and out.stride(1) == 1 and a.stride(1) == 1, "head_matmul: layout")
     H, N, K = w.shape
+    few = w.dtype == torch.bfloat16 and bool(lib().edgelm_head_matmul_few_takes(_p(a), a.stride(0), int(a_head_stride), _p(w), a.shape[0], K))
     _need((H - 1) * a_head_stride + K <= a.shape[1] and (H - 1) * out_head_stride + N <= out.shape[1] and out.shape[0] == a.shape[0], "head_matmul: shapes")
+    if few:      # (steps of few tokens: on the tensor cores, the activations as three bfloat16 terms)
+        _check(lib().edgelm_head_matmul_few(_p(a), a.stride(0), int(a_head_stride), _p(w), _p(out), _dt(out), out.stride(0), int(out_head_stride),
+                                            a.shape[0], H, K, N, _stream()))
+        return
     _check(lib().edgelm_head_matmul(_p(a), a.stride(0), int(a_head_stride), _p(w), _dt(w), _p(out), _dt(out), out.stride(0), int(out_head_stride),
                                     a.shape[0], H, K, N, _stream()))
 
@@ -873,6 +878,31 @@ def masked_attn_tiled(q, out, kcache, vcache, page_table, tile_seq, tile_tok0, t
                                           int(max_tile_tokens), nh, nkv, dk, dv, ctypes.c_float(scale), int(mask), int(mask_size or 0), _p(sink),
                                           int(n_splits), _p(part), T, int(maps), _p(gate), gate.stride(0) if gate is not None else 0, int(keep), gate_ch, _stream()),
            launches=2 if n_splits > 1 else 1)
+
+
+def latent_decode_takes(dtype, nh, dc, dv):
+    """How many of `nh` query heads a block of `latent_decode` takes together over rows of `dc` values of which the first `dv` are the
+    value (bfloat16 rows, sizes in steps of 16 that fit into a block's shared memory), or 0: not taken."""
+    return int(lib().edgelm_latent_decode_takes(int(nh), int(dc), int(dv))) if dtype == torch.bfloat16 else 0
+
+
+def latent_decode(q, out, kcache, tok_pos, tok_seq, page_table, nh, dc, dv, scale, mask, mask_size, sink, n_splits, part, gate=None, keep=0):
+    """Attention of one token a sequence over latent rows that are key and value at once (`masked_attn_tiled` with one key head and
+    `vcache` None) on the tensor cores, scores and weights in float32.  q [T, nh dc] float32, kcache [pages, 1, 64, dc] bfloat16, out
+    [T, nh dv] float32; `part`: float32, T nh n_splits (2 + dv) values, always needed."""
+    _f32(q, "q"); _f32(out, "out"); _f32(part, "part")
+    T = q.shape[0]
+    _need(q.shape == (T, nh * dc) and out.shape == (T, nh * dv) and part.numel() >= T * nh * n_splits * (2 + dv), "latent_decode: shapes")
+    _masked_cache_check(kcache, None, 1, dc, dv, "latent_decode")
+    _need(sink is None or (sink.dtype == torch.float32 and sink.is_contiguous() and sink.numel() == nh), "latent_decode: sink")
+    _need(gate is None or (gate.dtype == torch.float32 and gate.is_cuda and gate.shape == (T, nh) and gate.stride(1) == 1), "latent_decode: the heads' gate")
+    _need(latent_decode_takes(kcache.dtype, nh, dc, dv) > 0, "latent_decode: these sizes are not taken")
+    for t, n in ((tok_pos, "tok_pos"), (tok_seq, "tok_seq"), (page_table, "page_table")):
+        _i32(t, n)
+    _check(lib().edgelm_latent_decode(_p(q), _p(kcache), _p(tok_pos), _p(tok_seq), _p(page_table), page_table.stride(0), kcache.shape[0], T, nh, dc, dv,
+                                      ctypes.c_float(scale), int(mask), int(mask_size or 0), int(keep), int(n_splits), _p(part), _stream()))
+    _check(lib().edgelm_masked_attn_fold(_p(part), _p(out), _dt(out), _p(sink), T, nh, dv, int(n_splits), _p(gate),
+                                         gate.stride(0) if gate is not None else 0, _stream()))
 
 
 SPLIT_PREFILL_TILE = 64  # new tokens per tile of the split-precision tensor-core prefill kernel (SP_ROWS in attention_mma_split.cu)

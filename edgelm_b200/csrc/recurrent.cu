@@ -462,6 +462,49 @@ __global__ void rmsnorm_add_kernel(float* __restrict__ x, const float* __restric
   }
 }
 
+// The same for rows of whole 16-byte pieces, up to MAXV of them a thread: the row stays in registers between its sum of squares
+// and the scaling, and x and the weights are on their way while the sum is made.
+template <typename TCast, int MAXV>
+__global__ void __launch_bounds__(1024)
+rmsnorm_add_vec_kernel(float* __restrict__ x, const float* __restrict__ y1, float a, const float* __restrict__ y2, float b,
+                       const float* __restrict__ w, TCast* __restrict__ xc, int dim, float eps) {
+  pdl_launch_dependents();
+  __shared__ float red[33];
+  const int pieces = dim >> 2;
+  float4 g[MAXV], v[MAXV], xv[MAXV];
+#pragma unroll
+  for (int j = 0; j < MAXV; ++j) {      // (nothing on the stream writes the weights: they are read ahead of the wait)
+    const int i = threadIdx.x + j * blockDim.x;
+    if (i < pieces) g[j] = reinterpret_cast<const float4*>(w)[i];
+  }
+  pdl_wait();
+  const size_t row = (size_t)blockIdx.x * dim;
+  float ss = 0.f;
+#pragma unroll
+  for (int j = 0; j < MAXV; ++j) {
+    const int i = threadIdx.x + j * blockDim.x;
+    if (i >= pieces) continue;
+    v[j] = reinterpret_cast<const float4*>(y1 + row)[i];
+    xv[j] = reinterpret_cast<const float4*>(x + row)[i];
+    v[j].x *= a; v[j].y *= a; v[j].z *= a; v[j].w *= a;
+    if (y2) {
+      const float4 u = reinterpret_cast<const float4*>(y2 + row)[i];
+      v[j].x = fmaf(b, u.x, v[j].x); v[j].y = fmaf(b, u.y, v[j].y); v[j].z = fmaf(b, u.z, v[j].z); v[j].w = fmaf(b, u.w, v[j].w);
+    }
+    ss = fmaf(v[j].x, v[j].x, ss); ss = fmaf(v[j].y, v[j].y, ss); ss = fmaf(v[j].z, v[j].z, ss); ss = fmaf(v[j].w, v[j].w, ss);
+  }
+  ss = block_sum(ss, red);
+  const float inv = 1.0f / sqrtf(ss / (float)dim + eps);
+#pragma unroll
+  for (int j = 0; j < MAXV; ++j) {
+    const int i = threadIdx.x + j * blockDim.x;
+    if (i >= pieces) continue;
+    const float4 n = make_float4(xv[j].x + v[j].x * inv * g[j].x, xv[j].y + v[j].y * inv * g[j].y, xv[j].z + v[j].z * inv * g[j].z, xv[j].w + v[j].w * inv * g[j].w);
+    reinterpret_cast<float4*>(x + row)[i] = n;
+    if (xc) store_piece(xc + row + 4 * i, n);
+  }
+}
+
 // out = a y1 + b y2, or with `add` out += a y1 + b y2
 __global__ void scaled_sum_kernel(const float* __restrict__ y1, float a, const float* __restrict__ y2, float b, float* __restrict__ out, size_t n, int add) {
   pdl_launch_dependents();
@@ -636,6 +679,20 @@ extern "C" int edgelm_rmsnorm_add(float* x, const float* y1, float a, const floa
                                   int n_tokens, int dim, float eps, cudaStream_t stream) {
   if (n_tokens == 0) return 0;
   EL_REFUSE(n_tokens > 0 && dim > 0, "rmsnorm_add: bad sizes");
+  const bool vec = dim % 4 == 0 && dim <= 16384 && (uintptr_t)x % 16 == 0 && (uintptr_t)y1 % 16 == 0 && (uintptr_t)y2 % 16 == 0 && (uintptr_t)w % 16 == 0 && (uintptr_t)xc % 16 == 0;
+  if (vec) {
+    const int pieces = dim / 4, most = n_tokens <= 64 ? 1024 : (pieces <= 2048 ? 256 : 512), threads = pieces < most ? (pieces + 31) / 32 * 32 : most;
+    const int per = (pieces + threads - 1) / threads, bit = pdl_bit_for_tokens(n_tokens);
+#define EL_RA(TC, V) launch_pdl(bit, rmsnorm_add_vec_kernel<TC, V>, dim3(n_tokens), dim3(threads), (size_t)0, stream, x, y1, a, y2, b, w, (TC*)xc, dim, eps)
+#define EL_RAV(TC) do { if (per <= 1) EL_RA(TC, 1); else if (per <= 2) EL_RA(TC, 2); else if (per <= 4) EL_RA(TC, 4); else EL_RA(TC, 8); } while (0)
+    if (xc == nullptr || cast_dtype == DT_F32) EL_RAV(float);
+    else if (cast_dtype == DT_BF16) EL_RAV(__nv_bfloat16);
+    else EL_REFUSE(false, "rmsnorm_add: unknown dtype code %d", cast_dtype);
+#undef EL_RAV
+#undef EL_RA
+    EL_LAUNCH_CHECK("rmsnorm_add");
+    return 0;
+  }
   const dim3 grid(n_tokens), block(row_threads(dim));
   if (xc == nullptr || cast_dtype == DT_F32) launch_pdl(pdl_bit_for_tokens(n_tokens), rmsnorm_add_kernel<float>, dim3(grid), dim3(block), (size_t)(0), stream, x, y1, a, y2, b, w, (float*)xc, dim, eps);
   else if (cast_dtype == DT_BF16) launch_pdl(pdl_bit_for_tokens(n_tokens), rmsnorm_add_kernel<__nv_bfloat16>, dim3(grid), dim3(block), (size_t)(0), stream, x, y1, a, y2, b, w, (__nv_bfloat16*)xc, dim, eps);

@@ -31,7 +31,7 @@ from ..config.base import ConfigError
 from ..csrc import ops
 from . import linear
 from .base import KVNeed, Part, as_matrix, as_vector, nbytes
-from .masked_attention import MASKS, SHARED_KEYS_MIN_GROUP, decode_splits, kept_first, most_keys, read_mask, single_token_tiles, splits_room
+from .masked_attention import MASKS, MAX_SPLITS, SHARED_KEYS_MIN_GROUP, decode_splits, kept_first, most_keys, read_mask, single_token_tiles, splits_room
 from .registry import register_mixer
 from .rope import rotary_frequencies, rotary_magnitude
 
@@ -146,6 +146,13 @@ class LatentAttention(Part):
                 (nbytes((n_tokens, self.q_rank), self.dtype) + nbytes((n_tokens, self.nh * self.dq), f32) if self.q_rank else 0) + max(absorbed + splits_room(n_seqs, self.nh, self.rank), expanded) +
                 nbytes((n_tokens, self.nh * self.dv), self.dtype) + nbytes((n_tokens, self.hidden), self.dtype))
 
+    def _decode_splits(self, ctx, heads):
+        """Blocks that share a token's pages in `latent_decode`: as many as fill the device once, at most a block a page of the mask."""
+        splits = max(1, min(MAX_SPLITS, ctx.n_sms // max(1, ctx.n_seqs * -(-self.nh // heads))))
+        if self.mask != ops.MASK_CAUSAL:
+            splits = min(splits, (self.mask_size + 63) // 64 + 1 + (self.keep + 63) // 64)
+        return splits
+
     def _prepare(self, ctx, u, cache, q_out, q_pitch, q_off, copy_q, rows=None):
         """Queries from their latent if they have one; rotation; the latent's norm and the cache append (and the step's `rows`).
         q_out receives the queries' rotated part at q_off of every q_pitch values, with `copy_q` the unrotated part ahead of it.
@@ -222,7 +229,13 @@ class LatentAttention(Part):
         ol = ws.alloc((T, self.nh * self.rank), f32)
         tiled = ops.masked_attn_tiled_takes(self.dc, self.rank, own_values=False)      # (rows that a block can stage a page of)
         with ctx.prof("attn_latent"):
-            if ctx.all_single and self.nh >= SHARED_KEYS_MIN_GROUP and tiled:     # a row of the latent is staged once for all the heads
+            heads = ops.latent_decode_takes(self.dtype, self.nh, self.dc, self.rank) if ctx.all_single else 0
+            if heads:       # single tokens on the tensor cores: a row of the latent is staged once, as key and as value, for up to 32 heads
+                splits = self._decode_splits(ctx, heads)
+                part = ws.alloc((T * self.nh * splits * (2 + self.rank),), f32)
+                ops.latent_decode(qf, ol, cache.k, ctx.tok_pos, ctx.tok_seq, table, self.nh, self.dc, self.rank, self.scale, self.mask, self.mask_size,
+                                  self.sink, splits, part, gate=gate, keep=self.keep)
+            elif ctx.all_single and self.nh >= SHARED_KEYS_MIN_GROUP and tiled:     # a row of the latent is staged once for all the heads
                 splits = decode_splits(ctx, 1, self.nh, self.mask, self.mask_size, self.keep)
                 part = ws.alloc((T * self.nh * splits * (2 + self.rank),), f32) if splits > 1 else None
                 tseq, ttok0, tntok, tpos0 = single_token_tiles(ctx)

@@ -89,7 +89,29 @@ def _sarizen(vocab, width, ff, groups_of_layers, heads, kv_rank, rot_dim, window
             "layers": layers}
 
 
+def _semadra(vocab, width, ff, groups_of_layers, heads, kv_heads, q_rank, kv_rank, window, keep, side, experts, expert_ff, shared_ff):
+    """A Semadra-shaped model: per group a layer of attention, one of latent attention, one of latent attention over the latent that
+    the one before kept, and a second layer of attention, heads of 64, sliding windows (with kept first keys in the attention
+    layers); the first layer of all has the dense feed-forward, the others `experts` experts in four groups, two chosen out of the
+    two better groups, and a shared expert; every layer takes `side` numbers of the token's own in."""
+    moe = {"kind": "moe", "expert": {"ff": expert_ff}, "router": {"experts": experts, "top": 2, "groups": {"count": 4, "keep": 2}, "scale": 1.5},
+           "shared": {"ff": shared_ff}}
+    att = {"type": "attention", "mlp": moe, "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": 64, "vdim": 64, "scale": 0.125,
+                                                      "mask": {"size": window, "keep_first": keep}}}
+    lat = {"heads": heads, "dim": 64, "vdim": 64, "q_rank": q_rank, "kv_rank": kv_rank, "scale": 0.125, "mask": {"size": window}}
+    layers = []
+    for g in range(groups_of_layers):
+        layers += [att, {"type": "latent_attention", "mlp": moe, "mixer": lat},
+                   {"type": "latent_attention", "mlp": moe, "mixer": {**lat, "kv_from": 4 * g + 1}}, att]
+    layers[0] = {**att, "mlp": {"kind": "dense", "ff": ff}}
+    return {"architecture": "Semadra", "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "embedding": {"scale": width ** 0.5},
+            "residual_mult": 0.5, "token_side": {"dim": side}, "max_positions": 8192, "layers": layers}
+
+
 PRESETS = {
+    # the layer sizes of smollm2-135m and smollm2-1.7b (width, feed-forward, heads of 64, vocabulary) in the Semadra design
+    "semadra-576": _semadra(49152, 576, 1536, 2, 9, 3, 256, 128, 1024, 32, 64, 8, 768, 768),
+    "semadra-2048": _semadra(49152, 2048, 8192, 1, 32, 32, 1024, 512, 1024, 32, 256, 8, 4096, 4096),
     # the layer sizes of smollm2-135m and smollm2-1.7b (width, feed-forward, as many heads of 64, vocabulary) in the Sarizen design
     "sarizen-576": _sarizen(49152, 576, 1536, 2, 9, 128, 32, 1024, 8, 768, 768),
     "sarizen-2048": _sarizen(49152, 2048, 8192, 1, 32, 512, 64, 1024, 8, 4096, 4096),

@@ -151,3 +151,32 @@ def load(model_dir):
     with open(os.path.join(model_dir, "config.json")) as f:
         cfg = json.load(f)
     return cfg, read_safetensors(os.path.join(model_dir, "model.safetensors"))
+
+
+def closest_call(cfg, w, tokens):
+    """The smallest distance, over the tokens and the routers, between a chosen score (or a kept group's worth) and the first left-out one."""
+    side = cfg.get("token_side")
+    least, seen = 1.0, []
+
+    def watch(h, w_, mlp, pre, inner=moe_ffn):
+        seen.append((sigmoid(h @ w_[pre + "router"].T), mlp["router"]))
+        return inner(h, w_, mlp, pre)
+    keep = globals()["moe_ffn"]
+    globals()["moe_ffn"] = watch
+    try:
+        forward(cfg, w, tokens)
+    finally:
+        globals()["moe_ffn"] = keep
+    for s, r in seen:
+        groups = r.get("groups")
+        if groups:
+            parts = s.reshape(s.shape[0], groups["count"], -1)
+            worth = np.sort(np.sort(parts, axis=2)[:, :, ::-1][:, :, :2].sum(axis=2), axis=1)[:, ::-1]
+            if groups["keep"] < groups["count"]:
+                least = min(least, float((worth[:, groups["keep"] - 1] - worth[:, groups["keep"]]).min()))
+            order = np.argsort(-np.sort(parts, axis=2)[:, :, ::-1][:, :, :2].sum(axis=2), axis=1, kind="stable")[:, :groups["keep"]]
+            s = np.stack([parts[t, order[t]].reshape(-1) for t in range(len(s))])
+        if r["top"] < s.shape[1]:
+            s = np.sort(s, axis=1)[:, ::-1]
+            least = min(least, float((s[:, r["top"] - 1] - s[:, r["top"]]).min()))
+    return least
