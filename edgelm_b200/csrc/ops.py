@@ -813,6 +813,11 @@ def _gate_check(gate, T, nh, dv, what):
     return dv if gate is not None and dv > 1 and gate.shape[1] == nh * dv else 0
 
 
+def masked_attn_rows_takes(dtype, dk, dv, maps=1):
+    """Whether `masked_attn` reads whole key and value rows at a time for these heads (the rule of `launch_masked`)."""
+    return dtype == torch.bfloat16 and maps == 1 and dk % 8 == 0 and dv % 8 == 0 and dk <= 128 and dv <= 128
+
+
 def masked_attn(q, out, kcache, vcache, tok_pos, tok_seq, page_table, nh, nkv, dk, dv, scale, mask, mask_size, sink, max_keys, maps=1, gate=None,
                 n_splits=1, part=None, keep=0):
     """Attention of every token of the step over the keys lo .. its position (`mask`: MASK_CAUSAL lo = 0; MASK_WINDOW the

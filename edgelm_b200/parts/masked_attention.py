@@ -78,19 +78,21 @@ def most_keys(mask, size, keep=0):
 # keys are dealt to several such blocks and a second launch merges them (8 sequences of 32 heads of one to a key head: 254 ->
 # 143 us a layer), or, from SHARED_KEYS_LONG_GROUP heads to a key head on, the tiled kernel with its splits takes the step (9
 # heads of 3 to a key head: 72 us a layer against 85 with the pairs' keys dealt out; with one head to a key head it stages
-# every key for a tile of one row and loses, 254 against 183 us).
+# every key for a tile of one row and loses, 254 against 183 us).  The kernel that reads whole rows (`ops.masked_attn_rows_takes`) is
+# ahead of the tiled one at 3 heads to a key head too, and two of its blocks an SM are enough (9 heads of 3 to a key head over up to
+# 1,056 keys: a decode step 0.615 -> 0.594 ms; 32 heads of one to a key head: 0.675 ms with 4 blocks an SM, 0.659 with 2).
 SHARED_KEYS_MIN_GROUP = 8
 SPLIT_KEYS_FROM = 1024
 MAX_HEAD_SPLITS = 16
-BLOCKS_AN_SM = 4        # (8 sequences of 32 heads over 2,048 keys, a decode step: 0.722 ms with 2, 0.703 with 4, 0.717 with 8)
+BLOCKS_AN_SM, ROWS_BLOCKS_AN_SM = 4, 2        # (8 sequences of 32 heads over 2,048 keys, a decode step: 0.722 ms with 2, 0.703 with 4, 0.717 with 8)
 SHARED_KEYS_LONG_GROUP = 3
 
 
-def head_splits(ctx, n_pairs, mask, mask_size, keep=0):
-    """Blocks that share a (token, head) pair's keys in the block-per-pair kernel: about BLOCKS_AN_SM blocks of four warps an SM."""
+def head_splits(ctx, n_pairs, mask, mask_size, keep=0, an_sm=BLOCKS_AN_SM):
+    """Blocks that share a (token, head) pair's keys in the block-per-pair kernel: about `an_sm` blocks an SM."""
     if most_keys(mask, mask_size, keep) <= SPLIT_KEYS_FROM:
         return 1
-    return min(MAX_HEAD_SPLITS, max(1, (BLOCKS_AN_SM * ctx.n_sms + n_pairs - 1) // max(1, n_pairs)))
+    return min(MAX_HEAD_SPLITS, max(1, (an_sm * ctx.n_sms + n_pairs - 1) // max(1, n_pairs)))
 MAX_SPLITS = 32
 _ones = {}
 
@@ -189,6 +191,10 @@ class MaskedAttention(Part):
         """Whether prompt steps take the tensor-core kernel with float32 scores and weights (three bfloat16 terms for each
         float32 operand): one map a head, a bfloat16 cache, head sizes that it takes."""
         return self.maps == 1 and ops.attn_prefill_split_takes(self.dtype, self.dk, self.dv)
+
+    def _whole_rows(self):
+        """Whether the block-per-pair kernel of single tokens reads whole key and value rows at a time."""
+        return ops.masked_attn_rows_takes(self.dtype, self.dk, self.dv, self.maps)
 
     def tile_sizes(self):
         return (self.tile_tokens, ops.SPLIT_PREFILL_TILE) if self._on_tensor_cores() else (self.tile_tokens,)
@@ -314,14 +320,15 @@ class MaskedAttention(Part):
         with ctx.prof("attn_masked"):
             pairs = T * self.nh * self.maps
             long_and_few = ctx.all_single and most_keys(self.mask, self.mask_size, self.keep) > SPLIT_KEYS_FROM and pairs < 2 * ctx.n_sms
-            if ctx.all_single and (self.nh // self.nkv >= SHARED_KEYS_MIN_GROUP or (long_and_few and self.nh // self.nkv >= SHARED_KEYS_LONG_GROUP)):
+            if ctx.all_single and (self.nh // self.nkv >= SHARED_KEYS_MIN_GROUP or (long_and_few and self.nh // self.nkv >= SHARED_KEYS_LONG_GROUP and not self._whole_rows())):
                 splits = decode_splits(ctx, self.nkv * self.maps, self.nh // self.nkv, self.mask, self.mask_size, self.keep)
                 part = ws.alloc((T * self.nh * self.maps * splits * (2 + self.dv),), torch.float32) if splits > 1 else None
                 tseq, ttok0, tntok, tpos0 = single_token_tiles(ctx)
                 ops.masked_attn_tiled(q, a, cache.k, cache.v, table, tseq, ttok0, tntok, tpos0, T, 1, self.nh, self.nkv, self.dk, self.dv,
                                       self.scale, self.mask, self.mask_size, self.sink, n_splits=splits, part=part, maps=self.maps, gate=gate, keep=self.keep)
             elif ctx.all_single:
-                splits = head_splits(ctx, T * self.nh * self.maps, self.mask, self.mask_size, self.keep)
+                splits = head_splits(ctx, T * self.nh * self.maps, self.mask, self.mask_size, self.keep,
+                                     ROWS_BLOCKS_AN_SM if self._whole_rows() else BLOCKS_AN_SM)
                 part = ws.alloc((T * self.nh * self.maps * splits * (2 + self.dv),), torch.float32) if splits > 1 else None
                 ops.masked_attn(q, a, cache.k, cache.v, ctx.tok_pos, ctx.tok_seq, table, self.nh, self.nkv, self.dk, self.dv, self.scale,
                                 self.mask, self.mask_size, self.sink, most_keys(self.mask, self.mask_size, self.keep), maps=self.maps, gate=gate,
